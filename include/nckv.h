@@ -391,6 +391,61 @@ NCKV_API int nckv_glue_relu_sq(const void *h, void *out, int64_t n, void *stream
 NCKV_API int nckv_glue_ve_gate(const void *v, int64_t v_row_stride, const void *gate_lin, const void *ve, void *v_out, int rows, int Hkv, int D,
                       void *stream);
 
+/*
+ * Building blocks of decoders whose layers mix windowed attention and linear recurrences (registered in
+ * nanochat_b200/models.py).  `f32` selects fp32 activations instead of bf16; norms, positions, scores,
+ * recurrent states and the residual stream are fp32 in both.
+ *
+ * nckv_prefill_attn_split_p, nckv_decode_attn_split_p: nckv_prefill_attn / nckv_decode_attn with every
+ *   probability entering the product with V as two bf16 terms (16 bits of it).
+ * nckv_rope_unit_append: rotates the first rot_dims channels of q and k (pairs i, i + rot_dims / 2; cos_sin is
+ *   (rope_len, rot_dims) fp32, cosines then sines, any amplitude included), divides q and k by their root mean
+ *   square over Dk, multiplies q by q_scale; q -> q_out (B, T, Hq, Dk_pad), k and v -> the caches (token stride,
+ *   then heads of Dk_pad / Dv_pad channels) at cache_seqlens[b] + t.  Padding is written as zeros.  q, k, v are
+ *   rows of packed heads with their own row strides.
+ * nckv_window_attn: query at position p sees keys j with 0 <= p - j < window; any head size up to 512, fp32 math.
+ * nckv_recurrent: S <- diag(w) S + k v^T per head, state (B, H, Dk, Dv) fp32 read and updated in place.  With
+ *   `x` (rows of H * Dk fp32): w = exp(-exp(x + x0)) per token and channel and o = (S_prev + diag(u) k v^T)^T q;
+ *   else w = decay[h] and o = S^T q.  act_in: silu on q, k and v.  With norm_w: out = o / rms(o) * norm_w * silu(gate)
+ *   per head (needs x; Dv <= 128), of q's type; else out is o in fp32.  Dk <= 256.  Long prompts with few
+ *   (row, head) pairs need nckv_recurrent_workspace_bytes() of scratch (0: none).
+ * nckv_gated_norm: out = x / rms(x) * w * sigmoid(gate), or silu(gate), rms over groups of `group` channels.
+ * nckv_resid_norm: x' = x + y / rms(y) * w (or table[token]); x_out = x', h = x' or x' / rms(x') * final_w,
+ *   mix[m] = x' + (before - x') * mu[m] with the previous token's x' (carry holds it between calls, and is
+ *   updated).  x_out must not alias x when mix is given.
+ * nckv_silu_mul: rows [gate | up] of 2F -> silu(gate) * up.  nckv_tanh_split: tanh(z), fp32 or bf16 [hi | lo].
+ * nckv_softcap: z = cap * tanh(z / cap) in place.
+ */
+NCKV_API int nckv_prefill_attn_split_p(const void *q, const void *k, const void *v, const int32_t *cache_seqlens, void *out,
+                      int B, int T_new, int Hq, int Hkv, int D, int T_k, int64_t kv_batch_stride,
+                      int64_t kv_token_stride, int window_left, int32_t *status, void *stream);
+NCKV_API int nckv_decode_attn_split_p(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens,
+                      void *out, int B, int Hq, int Hkv, int D, int T_max, int64_t cache_batch_stride,
+                      int64_t cache_token_stride, int seqlen_offset, int window_left, void *workspace,
+                      size_t workspace_bytes, void *stream);
+NCKV_API int nckv_rope_unit_append(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *cos_sin, const int32_t *cache_seqlens, void *q_out, void *k_cache, void *v_cache,
+                      int64_t k_batch_stride, int64_t k_token_stride, int64_t v_batch_stride, int64_t v_token_stride,
+                      int B, int T, int Hq, int Hkv, int Dk, int Dv, int Dk_pad, int Dv_pad, int rot_dims, int rope_len,
+                      int T_max, float q_scale, float eps, int f32, int32_t *status, void *stream);
+NCKV_API int nckv_window_attn(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens, void *out,
+                      int64_t k_batch_stride, int64_t k_token_stride, int64_t v_batch_stride, int64_t v_token_stride, int B,
+                      int T, int Hq, int Hkv, int Dk, int Dv, int T_max, int window, float scale, int f32, void *stream);
+NCKV_API size_t nckv_recurrent_workspace_bytes(int B, int T, int H, int Dk, int Dv);
+NCKV_API int nckv_recurrent(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *x, int64_t x_stride, const float *x0, const float *u, const float *decay,
+                      const void *gate, int64_t gate_stride, const float *norm_w, float eps, void *out, int64_t out_stride,
+                      float *state, int B, int T, int H, int Dk, int Dv, int act_in, int f32, void *workspace,
+                      size_t workspace_bytes, void *stream);
+NCKV_API int nckv_gated_norm(const float *x, const void *gate, int64_t gate_stride, const float *w, void *out, int rows, int C,
+                      int group, float eps, int gate_silu, int f32, void *stream);
+NCKV_API int nckv_resid_norm(const float *x, const void *y, int y_f32, const float *w, const int64_t *tokens, const void *table,
+                      int vocab, float *x_out, void *h, const float *final_w, void *mix, const float *mu, int n_mix,
+                      float *carry, int B, int T, int W, float eps, int f32, void *stream);
+NCKV_API int nckv_silu_mul(const void *gate_up, void *out, int64_t rows, int F, int f32, void *stream);
+NCKV_API int nckv_tanh_split(const float *z, void *out, int64_t rows, int R, int f32, void *stream);
+NCKV_API int nckv_softcap(float *z, int64_t n, float cap, void *stream);
+
 #ifdef __cplusplus
 }
 #endif

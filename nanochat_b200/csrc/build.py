@@ -4,15 +4,19 @@ Usage:  python -m nanochat_b200.csrc.build [--verbose] [--force]
 The shared library is written next to the package (nanochat_b200/libnckv.so); it is a build
 artefact and is not tracked.
 """
+import fcntl
 import os
 import subprocess
 import sys
+import tempfile
+from concurrent.futures import ThreadPoolExecutor
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 PKG = os.path.dirname(HERE)
 OUT = os.path.join(PKG, "libnckv.so")
 SOURCES = ["host.cu", "append.cu", "decode_attn.cu", "prefill_broadcast.cu", "lse_combine.cu",
-           "prefill_attn.cu", "p2p_exchange.cu", "glue.cu", "flash_attn_bwd.cu", "host_step.cu"]
+           "prefill_attn.cu", "p2p_exchange.cu", "glue.cu", "flash_attn_bwd.cu", "host_step.cu",
+           "recurrent.cu", "norm_mix.cu", "window_attn.cu"]
 HEADERS = ["nckv_common.cuh", "tc05.cuh", os.path.join("..", "..", "include", "nckv.h")]
 
 
@@ -31,21 +35,34 @@ def up_to_date():
     return all(os.path.getmtime(d) <= t for d in deps)
 
 
-def build(verbose=False, force=False):
-    if not force and up_to_date():
-        return OUT
-    cmd = [_nvcc(), "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-           "--shared", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
-           "-o", OUT] + [os.path.join(HERE, s) for s in SOURCES]
-    if verbose:
-        cmd.insert(1, "-Xptxas")
-        cmd.insert(2, "-v")
-        print(" ".join(cmd), flush=True)
+def _compile(cmd, verbose):
     res = subprocess.run(cmd, capture_output=True, text=True)
     if verbose or res.returncode != 0:
-        sys.stderr.write(res.stdout + res.stderr)
-    if res.returncode != 0:
-        raise RuntimeError("nvcc failed building libnckv.so")
+        sys.stderr.write(" ".join(cmd) + "\n" + res.stdout + res.stderr)
+    return res.returncode
+
+
+def build(verbose=False, force=False):
+    """Compile the sources side by side, link them, and move the library into place in one step; several
+    processes may call this at the same time."""
+    if not force and up_to_date():
+        return OUT
+    with open(os.path.join(PKG, ".build.lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not force and up_to_date():  # another process has built it meanwhile
+            return OUT
+        nvcc = _nvcc()
+        flags = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC",
+                 "-Xcompiler", "-fvisibility=hidden"] + (["-Xptxas", "-v"] if verbose else [])
+        with tempfile.TemporaryDirectory(dir=PKG, prefix=".build-") as tmp:
+            objs = [os.path.join(tmp, os.path.splitext(s)[0] + ".o") for s in SOURCES]
+            jobs = [[nvcc] + flags + ["-c", "-o", o, os.path.join(HERE, s)] for s, o in zip(SOURCES, objs)]
+            with ThreadPoolExecutor(max(1, min(len(jobs), os.cpu_count() or 1))) as pool:
+                failed = any(list(pool.map(lambda cmd: _compile(cmd, verbose), jobs)))
+            linked = os.path.join(tmp, os.path.basename(OUT))
+            if failed or _compile([nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "--shared", "-o", linked] + objs, verbose):
+                raise RuntimeError("nvcc failed building libnckv.so")
+            os.replace(linked, OUT)
     return OUT
 
 

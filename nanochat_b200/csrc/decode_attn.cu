@@ -22,7 +22,8 @@
 // Math per tile.  All G = Hq/Hkv query heads that share a kv head are the rows of one
 // m16n8k16 tile (rows >= G are zero), so K/V bytes are read once per group.  S = Q K^T and
 // O += P V use the warp-level bf16 MMA with fp32 accumulation; running max / sum use quad
-// shuffles; P is rounded to bf16 for the second product, as the flash-style library kernels do.
+// shuffles; P is rounded to bf16 for the second product, as the flash-style library kernels do (the
+// SPLIT_P form multiplies V by two bf16 terms of P, which keeps 16 bits of every probability).
 //
 // Combine.  A pair whose tiles all fall inside one run is normalised and written directly.
 // Otherwise every run that touches the pair leaves an un-normalised partial (O, m, l) in the
@@ -292,7 +293,7 @@ __device__ __forceinline__ void page_coords(const DecodeParams &p, int b, int ke
 // GHI: group size 9..16 (rows 8..15 of the MMA tile carry heads too).  MAP5: the tensor maps are the
 // 5-D form (one copy per K or V tile) instead of the 4-D form (one copy per 64-channel half).
 // PAGED: block-table storage (always with the 5-D maps, whose outermost coordinate is then the page).
-template <bool GHI, bool MAP5, bool PAGED = false>
+template <bool GHI, bool MAP5, bool PAGED = false, bool SPLIT_P = false>
 __global__ void __launch_bounds__(DEC_WARPS * 32, DEC_CTAS_PER_SM)
 decode_attn_kernel(const __grid_constant__ CUtensorMap tmap_k,
                    const __grid_constant__ CUtensorMap tmap_v, const DecodeParams p) {
@@ -612,20 +613,23 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmap_k,
         m_run[0] = mn0;
         if (GHI) m_run[1] = mn1;
         float rs0 = 0.f, rs1 = 0.f;
-        uint32_t pa[DEC_TILE / 8][2];
+        uint32_t pa[DEC_TILE / 8][2], pl[SPLIT_P ? DEC_TILE / 8 : 1][2];
 #pragma unroll
         for (int nb = 0; nb < DEC_TILE / 8; ++nb) {
             const float p0 = exp2f(fmaf(s_acc[nb][0], p.scale_log2, -mn0));
             const float p1 = exp2f(fmaf(s_acc[nb][1], p.scale_log2, -mn0));
             rs0 += p0 + p1;
             pa[nb][0] = pack_bf16x2(p0, p1);
+            if constexpr (SPLIT_P) pl[nb][0] = pack_bf16x2(p0 - bf16lo(pa[nb][0]), p1 - bf16hi(pa[nb][0]));
             if (GHI) {
                 const float p2 = exp2f(fmaf(s_acc[nb][2], p.scale_log2, -mn1));
                 const float p3 = exp2f(fmaf(s_acc[nb][3], p.scale_log2, -mn1));
                 rs1 += p2 + p3;
                 pa[nb][1] = pack_bf16x2(p2, p3);
+                if constexpr (SPLIT_P) pl[nb][1] = pack_bf16x2(p2 - bf16lo(pa[nb][1]), p3 - bf16hi(pa[nb][1]));
             } else {
                 pa[nb][1] = 0u;
+                if constexpr (SPLIT_P) pl[nb][1] = 0u;
             }
         }
         l_run[0] = l_run[0] * alpha0 + rs0;  // per-lane partial sums; reduced over the quad at the end
@@ -651,6 +655,12 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                pa[2 * ks][0], pa[2 * ks][1], pa[2 * ks + 1][0], pa[2 * ks + 1][1], b0, b1);
                 mma_bf16_16816(o_acc[nd + 1][0], o_acc[nd + 1][1], o_acc[nd + 1][2], o_acc[nd + 1][3],
                                pa[2 * ks][0], pa[2 * ks][1], pa[2 * ks + 1][0], pa[2 * ks + 1][1], b2, b3);
+                if constexpr (SPLIT_P) {
+                    mma_bf16_16816(o_acc[nd][0], o_acc[nd][1], o_acc[nd][2], o_acc[nd][3],
+                                   pl[2 * ks][0], pl[2 * ks][1], pl[2 * ks + 1][0], pl[2 * ks + 1][1], b0, b1);
+                    mma_bf16_16816(o_acc[nd + 1][0], o_acc[nd + 1][1], o_acc[nd + 1][2], o_acc[nd + 1][3],
+                                   pl[2 * ks][0], pl[2 * ks][1], pl[2 * ks + 1][0], pl[2 * ks + 1][1], b2, b3);
+                }
             }
         }
 
@@ -1081,7 +1091,8 @@ static int decode_launch(const void *q, const void *k_cache, const void *v_cache
                          void *out, float *out_f32, float *lse_out, int B, int Hq, int Hkv, int D, int T_max,
                          int64_t cache_batch_stride, int64_t cache_token_stride, int seqlen_offset, int window_left,
                          int kv_begin, int kv_end, nckv::KvSplit split, const nckv::PushDesc &push, void *workspace,
-                         size_t workspace_bytes, void *stream, nckv::PagedDesc paged = nckv::PagedDesc{nullptr, 0, 0, 0}) {
+                         size_t workspace_bytes, void *stream, nckv::PagedDesc paged = nckv::PagedDesc{nullptr, 0, 0, 0},
+                         bool split_p = false) {
     using namespace nckv;
     int rc0 = decode_check(q, k_cache, v_cache, cache_seqlens, out, out_f32, workspace, B, Hq, Hkv, D, T_max,
                            workspace_bytes);
@@ -1152,13 +1163,21 @@ static int decode_launch(const void *q, const void *k_cache, const void *v_cache
         NCKV_CUDA_CHECK(cudaFuncSetAttribute(decode_attn_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max));
         NCKV_CUDA_CHECK(cudaFuncSetAttribute(decode_attn_kernel<true, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max));
         NCKV_CUDA_CHECK(cudaFuncSetAttribute(decode_attn_kernel<false, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max));
+        NCKV_CUDA_CHECK(cudaFuncSetAttribute(decode_attn_kernel<true, true, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max));
+        NCKV_CUDA_CHECK(cudaFuncSetAttribute(decode_attn_kernel<false, true, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max));
         attr_set[dev] = true;
+    }
+    if (split_p && (!map5 || paged.table)) {
+        set_error("decode_attn_split_p: needs a dense cache and a driver that accepts the 5-D tensor maps");
+        return NCKV_E_UNSUPPORTED;
     }
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     // Both launches allow programmatic overlap with their predecessor in the stream: each kernel
     // runs its set-up early and waits (griddepcontrol.wait) before it touches dependent data.
     const dim3 g3(grid), b3(DEC_WARPS * 32);
-    if (paged.table && ghi) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<true, true, true>, g3, b3, smem, s, true, mk, mv, p));
+    if (split_p && ghi) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<true, true, false, true>, g3, b3, smem, s, true, mk, mv, p));
+    else if (split_p) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<false, true, false, true>, g3, b3, smem, s, true, mk, mv, p));
+    else if (paged.table && ghi) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<true, true, true>, g3, b3, smem, s, true, mk, mv, p));
     else if (paged.table) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<false, true, true>, g3, b3, smem, s, true, mk, mv, p));
     else if (ghi && map5) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<true, true>, g3, b3, smem, s, true, mk, mv, p));
     else if (ghi) NCKV_CUDA_CHECK(launch_pdl(decode_attn_kernel<true, false>, g3, b3, smem, s, true, mk, mv, p));
@@ -1195,6 +1214,20 @@ int nckv_decode_attn(const void *q, const void *k_cache, const void *v_cache,
     return decode_launch(q, k_cache, v_cache, cache_seqlens, out, out_f32, lse_out, B, Hq, Hkv, D, T_max,
                          cache_batch_stride, cache_token_stride, seqlen_offset, window_left, kv_begin, kv_end,
                          nckv::KvSplit{0, 0, 0}, none, workspace, workspace_bytes, stream);
+}
+
+int nckv_decode_attn_split_p(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens, void *out,
+                             int B, int Hq, int Hkv, int D, int T_max, int64_t cache_batch_stride,
+                             int64_t cache_token_stride, int seqlen_offset, int window_left, void *workspace,
+                             size_t workspace_bytes, void *stream) {
+    if (!out) {
+        nckv::set_error("decode_attn_split_p: null pointer argument");
+        return NCKV_E_ARG;
+    }
+    nckv::PushDesc none = {};
+    return decode_launch(q, k_cache, v_cache, cache_seqlens, out, nullptr, nullptr, B, Hq, Hkv, D, T_max,
+                         cache_batch_stride, cache_token_stride, seqlen_offset, window_left, 0, 0,
+                         nckv::KvSplit{0, 0, 0}, none, workspace, workspace_bytes, stream, nckv::PagedDesc{nullptr, 0, 0, 0}, true);
 }
 
 int nckv_decode_attn_paged(const void *q, const void *k_pool, const void *v_pool, const int32_t *block_table,

@@ -24,6 +24,8 @@
 //                     grown by more than 2^8; only then is the O row rescaled in TMEM
 //                     (tcgen05.ld / multiply / tcgen05.st), so most tiles neither wait for nor
 //                     touch the accumulator.  O is read once, at the end.
+// The SPLIT_P form keeps the probabilities to 16 bits: P goes to TMEM as two bf16 terms, hi over the
+// first and lo over the last 32 columns of its S buffer, and O += P V becomes 8 products per tile.
 // Products issued by one thread execute in order: S of tile it+2 is issued behind O += P V(it)
 // and may therefore overwrite the buffer P(it) was read from.
 // Two CTAs fit on an SM (112 KB of shared memory and 256 of the 512 TMEM columns each), so one
@@ -139,6 +141,7 @@ struct PfCursor {
     __device__ __forceinline__ bool last_of_item() const { return t == it.n_tiles - 1; }
 };
 
+template <bool SPLIT_P>
 __global__ void __launch_bounds__(PF_THREADS, 2)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                     const __grid_constant__ CUtensorMap tmap_v, const PrefillParams p) {
@@ -324,9 +327,9 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
                 const uint64_t dv = desc_v + (uint64_t)((vstage * PF_KV_BYTES) >> 4);
                 const uint32_t pbase = tmem_s + (gp & 1u) * PF_N;
 #pragma unroll
-                for (int ks = 0; ks < PF_N / 16; ++ks) {
-                    // P(gp) sits in the first 32 columns of its S buffer; 16 keys = 8 columns
-                    const uint64_t db = dv + (uint64_t)((ks * 16 * 128) >> 4);
+                for (int ks = 0; ks < (SPLIT_P ? 2 : 1) * PF_N / 16; ++ks) {
+                    // P(gp) sits in the first 32 columns of its S buffer (its low terms in the next 32); 16 keys = 8 columns
+                    const uint64_t db = dv + (uint64_t)(((ks & (PF_N / 16 - 1)) * 16 * 128) >> 4);
                     umma_bf16_a_tmem(tmem_o, pbase + (uint32_t)ks * 8, db, IDESC_O, (pc.t > 0 || ks > 0) ? 1u : 0u);
                 }
                 // S(gp+2), issued behind this product into the S buffer P(gp) sits in, tells of its completion
@@ -416,7 +419,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
                 const float m_use = m_used == -INFINITY ? 0.f : m_used;  // a row that has seen no key yet
                 float2 rs01 = make_float2(0.f, 0.f), rs23 = make_float2(0.f, 0.f);
                 const float2 scale2 = make_float2(p.scale_log2, p.scale_log2), neg_m2 = make_float2(-m_use, -m_use);
-                uint32_t pk[PF_N / 2];
+                uint32_t pk[PF_N / 2], pk_lo[SPLIT_P ? PF_N / 2 : 1];
 #pragma unroll
                 for (int c = 0; c < PF_N; c += 4) {
                     // 2^(s * scale - m): one two-wide FFMA per pair of scores, one MUFU.EX2 per score
@@ -428,12 +431,17 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
                     rs23 = fadd2(rs23, p23);
                     pk[c / 2] = pack_bf16x2(p01.x, p01.y);
                     pk[c / 2 + 1] = pack_bf16x2(p23.x, p23.y);
+                    if constexpr (SPLIT_P) {
+                        pk_lo[c / 2] = pack_bf16x2(p01.x - bf16lo(pk[c / 2]), p01.y - bf16hi(pk[c / 2]));
+                        pk_lo[c / 2 + 1] = pack_bf16x2(p23.x - bf16lo(pk[c / 2 + 1]), p23.y - bf16hi(pk[c / 2 + 1]));
+                    }
                 }
                 l_run += (rs01.x + rs01.y) + (rs23.x + rs23.y);
 
                 // P row -> TMEM, over the first 32 columns of this tile's S buffer (this lane's own scores,
                 // already in registers).  S of tile g+2 is issued behind P V(g) and lands on top of it.
                 tmem_st_words(tmem_s_it + lane_sel, pk);
+                if constexpr (SPLIT_P) tmem_st_words(tmem_s_it + 32 + lane_sel, pk_lo);
                 // A raised scale: O (+)= P V of the previous tile must be complete before the O rows
                 // accumulated so far are brought to the new scale (tcgen05.ld / multiply / tcgen05.st).
                 // Every lane applies its own factor (1 for rows that keep their scale).
@@ -529,8 +537,10 @@ static size_t prefill_smem_bytes() {
 
 static int prefill_launch(const void *q, const void *k, const void *v, const int32_t *cache_seqlens, void *out,
                           float *lse, int B, int T_new, int Hq, int Hkv, int D, int T_k, int64_t kv_batch_stride,
-                          int64_t kv_token_stride, int window_left, int32_t *status, void *stream) {
+                          int64_t kv_token_stride, int window_left, int32_t *status, void *stream,
+                          bool split_p = false) {
     using namespace nckv;
+    const auto kernel = split_p ? prefill_attn_kernel<true> : prefill_attn_kernel<false>;
     if (!q || !k || !v || !out || !status) {
         set_error("prefill_attn: null pointer argument");
         return NCKV_E_ARG;
@@ -611,7 +621,8 @@ static int prefill_launch(const void *q, const void *k, const void *v, const int
     int dev = 0;
     NCKV_CUDA_CHECK(cudaGetDevice(&dev));
     if (dev < 64 && !attr_set[dev]) {
-        NCKV_CUDA_CHECK(cudaFuncSetAttribute(prefill_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        NCKV_CUDA_CHECK(cudaFuncSetAttribute(prefill_attn_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        NCKV_CUDA_CHECK(cudaFuncSetAttribute(prefill_attn_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         attr_set[dev] = true;
     }
     cudaLaunchConfig_t cfg = {};
@@ -624,7 +635,7 @@ static int prefill_launch(const void *q, const void *k, const void *v, const int
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    NCKV_CUDA_CHECK(cudaLaunchKernelEx(&cfg, prefill_attn_kernel, mq, mk, mv, p));
+    NCKV_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, mq, mk, mv, p));
     return NCKV_OK;
 }
 
@@ -634,6 +645,14 @@ extern "C" int nckv_prefill_attn(const void *q, const void *k, const void *v, co
                                  int32_t *status, void *stream) {
     return prefill_launch(q, k, v, cache_seqlens, out, nullptr, B, T_new, Hq, Hkv, D, T_k, kv_batch_stride,
                           kv_token_stride, window_left, status, stream);
+}
+
+extern "C" int nckv_prefill_attn_split_p(const void *q, const void *k, const void *v, const int32_t *cache_seqlens,
+                                         void *out, int B, int T_new, int Hq, int Hkv, int D, int T_k,
+                                         int64_t kv_batch_stride, int64_t kv_token_stride, int window_left,
+                                         int32_t *status, void *stream) {
+    return prefill_launch(q, k, v, cache_seqlens, out, nullptr, B, T_new, Hq, Hkv, D, T_k, kv_batch_stride,
+                          kv_token_stride, window_left, status, stream, true);
 }
 
 // Forward of flash_attn_func for training: the same kernel over plain (B, T, H, D) tensors, which also

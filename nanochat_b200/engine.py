@@ -1,4 +1,6 @@
-"""KV cache with the reference's interface (nanochat/engine.py:82-137), storage on the GPU.
+"""Caches, sampling and the generation loop.
+
+KV cache with the reference's interface (nanochat/engine.py:82-137), storage on the GPU.
 
 ``KVCache`` keeps the reference's constructor, attributes (``k_cache`` / ``v_cache`` of shape
 (n_layers, B, T_max, Hkv, D), int32 ``cache_seqlens``, ``prev_embedding``) and methods
@@ -50,6 +52,11 @@ class KVCache:
     def advance(self, num_tokens):
         """cache_seqlens += num_tokens for every row (engine.py:119-121)."""
         self.cache_seqlens += num_tokens
+
+    @property
+    def capturable(self):
+        """Whether a decode step over this cache can be captured in a CUDA graph yet."""
+        return self.prev_embedding is not None
 
     def prefill(self, other):
         """Broadcast a batch-1 prompt cache into every row of this (empty) cache (engine.py:123-137).
@@ -132,6 +139,8 @@ class PagedKVCache:
     def advance(self, num_tokens):
         self.cache_seqlens += num_tokens
 
+    capturable = KVCache.capturable
+
     # ---- page bookkeeping (host) ---------------------------------------------------------------
     def pages_in_use(self):
         return self.n_pages - len(self._free)
@@ -192,6 +201,119 @@ class PagedKVCache:
         self.cache_seqlens.fill_(p)
         if other.prev_embedding is not None:
             self.prev_embedding = other.prev_embedding.expand(B, -1, -1).clone()
+
+
+class HybridCache:
+    """What a decoder with several kinds of layers keeps per sequence, behind KVCache's methods.
+
+    Layers declare their parts by name: ``add_kv`` a pair of dense (B, T_max, heads, width) key and value
+    rows, ``add_state`` a fixed-size fp32 state per row (recurrent states, carried vectors), ``add_table``
+    a constant table over positions (one per key, shared by the layers that ask for it, built by the
+    first).  Key and value rows are written before they are read and need no clearing; states start at
+    zero, so ``reset`` clears them.  All rows of a batch move through ``cache_seqlens`` like KVCache's."""
+
+    capturable = True  # a step over it can be captured in a CUDA graph from the start
+
+    def __init__(self, batch_size, seq_len, device):
+        self.batch_size = batch_size
+        self.max_seq_len = seq_len
+        self.device = device
+        self.cache_seqlens = torch.zeros(batch_size, dtype=torch.int32, device=device)
+        self.kv, self.state, self.tables = {}, {}, {}
+
+    # ---- what layers keep ----------------------------------------------------------------------
+    def add_kv(self, key, heads, k_width, v_width, dtype):
+        # not zero-filled: nothing beyond cache_seqlens is ever attended
+        self.kv[key] = tuple(torch.empty(self.batch_size, self.max_seq_len, heads, width, dtype=dtype, device=self.device)
+                             for width in (k_width, v_width))
+
+    def add_state(self, key, shape):
+        self.state[key] = torch.zeros(self.batch_size, *shape, dtype=torch.float32, device=self.device)
+
+    def add_table(self, key, make):
+        if key not in self.tables:
+            self.tables[key] = make(self.max_seq_len, self.device)
+
+    def state_tensors(self):
+        """Everything a step changes in place, apart from the rows it appends."""
+        return [self.cache_seqlens, *self.state.values()]
+
+    # ---- KVCache's methods ---------------------------------------------------------------------
+    def reset(self):
+        for t in self.state_tensors():
+            t.zero_()
+
+    def get_pos(self):
+        return int(self.cache_seqlens[0].item())
+
+    def advance(self, num_tokens):
+        self.cache_seqlens += num_tokens
+
+    def prefill(self, other):
+        """Broadcast a batch-1 prompt cache into every row of this (empty) cache."""
+        assert self.get_pos() == 0, "Cannot prefill a non-empty cache"
+        assert other.batch_size == 1 and self.max_seq_len >= other.max_seq_len
+        assert self.kv.keys() == other.kv.keys() and self.state.keys() == other.state.keys()
+        p = other.get_pos()
+        for key, (k, v) in self.kv.items():
+            src_k, src_v = other.kv[key]
+            if k.shape == v.shape and k.dtype == torch.bfloat16 and k.size(3) == ops.HEAD_DIM:
+                ops.prefill_broadcast(src_k[None], src_v[None], k[None], v[None], None, p)
+            else:
+                k[:, :p].copy_(src_k[:, :p].expand(self.batch_size, -1, -1, -1))
+                v[:, :p].copy_(src_v[:, :p].expand(self.batch_size, -1, -1, -1))
+        for key, t in self.state.items():
+            t.copy_(other.state[key].expand_as(t))
+        self.cache_seqlens.fill_(p)
+
+
+class SequenceRunner:
+    """Runs portions of live sequences through a model, one entry at a time, each from what its earlier
+    portions left.  Caches of finished sequences are cleared and used again."""
+
+    def __init__(self, model, max_tokens):
+        self.model, self.max_tokens = model, max(int(max_tokens), 1)
+        self._live, self._free = {}, []
+
+    def feed(self, seq_id, tokens, want):
+        """Run ``tokens`` of the sequence; fp32 logits (len(want), vocab) at the places ``want``, or None."""
+        cache = self._live.get(seq_id)
+        if cache is None:
+            cache = self._free.pop() if self._free else new_cache(self.model, 1, self.max_tokens, torch.bfloat16)
+            self._live[seq_id] = cache
+        if not tokens:
+            return None
+        ids = torch.tensor([tokens], dtype=torch.long, device=self.model.get_device())
+        logits = forward_at(self.model, ids, cache, list(want))
+        return logits[0] if want else None
+
+    def finish(self, seq_id):
+        """Give back what the sequence holds."""
+        cache = self._live.pop(seq_id, None)
+        if cache is not None:
+            cache.reset()
+            self._free.append(cache)
+
+
+def forward_at(model, ids, cache, places):
+    """Logits (B, len(places), vocab) at the given places of the new tokens ``ids`` (B, T); models that can
+    skip the output head elsewhere do."""
+    if getattr(model, "accepts_logits_at", False):
+        return model.forward(ids, kv_cache=cache, logits_at=places)
+    return model.forward(ids, kv_cache=cache)[:, places]
+
+
+def new_cache(model, batch_size, seq_len, dtype, page_tokens=None, n_pages=None):
+    """An empty cache for ``model``: its own (``make_cache``) or, for any model with the reference's GPT
+    configuration, dense or paged key/value storage."""
+    if hasattr(model, "make_cache"):
+        return model.make_cache(batch_size, seq_len, page_tokens=page_tokens, n_pages=n_pages)
+    cfg = model.config
+    geometry = dict(num_heads=cfg.n_kv_head, head_dim=cfg.n_embd // cfg.n_head, num_layers=cfg.n_layer)
+    if page_tokens:
+        return PagedKVCache(batch_size=batch_size, seq_len=seq_len, device=model.get_device(), dtype=dtype,
+                            page_tokens=page_tokens, n_pages=n_pages, **geometry)
+    return KVCache(batch_size=batch_size, seq_len=seq_len, device=model.get_device(), dtype=dtype, **geometry)
 
 
 # ------------------------------------------------------------------------------------------------
@@ -290,20 +412,19 @@ class Engine:
         bos = self.tokenizer.get_bos_token_id()
 
         cfg = self.model.config
-        geometry = dict(num_heads=cfg.n_kv_head, head_dim=cfg.n_embd // cfg.n_head, num_layers=cfg.n_layer)
-        prompt_cache = KVCache(batch_size=1, seq_len=len(tokens), device=device, dtype=dtype, **geometry)
+        prompt_cache = new_cache(self.model, 1, len(tokens), dtype)
         ids = torch.tensor([tokens], dtype=torch.long, device=device)
-        logits = self.model.forward(ids, kv_cache=prompt_cache)[:, -1, :].expand(num_samples, -1)
+        logits = forward_at(self.model, ids, prompt_cache, [len(tokens) - 1])[:, -1, :].expand(num_samples, -1)
 
         capacity = (len(tokens) + max_tokens) if max_tokens is not None else cfg.sequence_len
         if self.page_tokens:
             # shared prompt pages + per row the pages its own continuation can need
             pt = self.page_tokens
             own = -(-capacity // pt) - len(tokens) // pt
-            cache = PagedKVCache(batch_size=num_samples, seq_len=capacity, device=device, dtype=dtype, page_tokens=pt,
-                                 n_pages=len(tokens) // pt + num_samples * own, **geometry)
+            cache = new_cache(self.model, num_samples, capacity, dtype, page_tokens=pt,
+                              n_pages=len(tokens) // pt + num_samples * own)
         else:
-            cache = KVCache(batch_size=num_samples, seq_len=capacity, device=device, dtype=dtype, **geometry)
+            cache = new_cache(self.model, num_samples, capacity, dtype)
         cache.prefill(prompt_cache)
         del prompt_cache
 
@@ -325,7 +446,7 @@ class Engine:
                 # and only pays off if enough steps are still to come
                 room = capacity - (len(tokens) + n_done)
                 left = (max_tokens - n_done) if max_tokens is not None else room
-                if room >= 4 and left >= 16 and cache.prev_embedding is not None:
+                if room >= 4 and left >= 16 and cache.capturable:
                     graphed = GraphedDecodeStep(self.model, cache, ids)
             if graphed is not None:
                 return graphed.step(ids)
@@ -411,8 +532,10 @@ class GraphedDecodeStep:
     captured (``get_pos()`` / ``.item()`` per forward and per layer, gpt.py:424, flash_attention.py:157).
 
     ``step(ids)`` copies the token ids into the graph's input buffer, replays, and returns the
-    logits buffer (B, vocab) — overwritten by the next call.  The smear state
-    (``kv_cache.prev_embedding``) is kept in a persistent buffer that the graph reads and updates.
+    logits buffer (B, vocab) — overwritten by the next call.  The smear state of a KVCache
+    (``kv_cache.prev_embedding``) is kept in a persistent buffer that the graph reads and updates; a
+    HybridCache's states are updated in place.  Warm-up and capture do not move the cache forward:
+    lengths and states are put back afterwards.
     """
 
     def __init__(self, model, kv_cache, warmup_ids):
@@ -420,12 +543,15 @@ class GraphedDecodeStep:
         self.model, self.cache = model, kv_cache
         dev = warmup_ids.device
         self.ids = warmup_ids.clone()
-        if kv_cache.prev_embedding is None:
+        if not kv_cache.capturable:
             raise RuntimeError("capture after the prefill forward: the cache has no smear state yet")
-        self._prev = kv_cache.prev_embedding.clone()
-        kv_cache.prev_embedding = self._prev
-        # capture must not move the real cache forward: remember lengths, restore after warm-up/capture
-        saved_lens = kv_cache.cache_seqlens.clone()
+        in_place = kv_cache.state_tensors() if hasattr(kv_cache, "state_tensors") else [kv_cache.cache_seqlens]
+        self._prev = None
+        if getattr(kv_cache, "prev_embedding", None) is not None:
+            self._prev = kv_cache.prev_embedding.clone()
+            kv_cache.prev_embedding = self._prev
+            in_place.append(self._prev)
+        saved = [t.clone() for t in in_place]
         side = torch.cuda.Stream(dev)
         side.wait_stream(torch.cuda.current_stream(dev))
         with torch.cuda.stream(side):
@@ -436,16 +562,16 @@ class GraphedDecodeStep:
             with torch.cuda.graph(self.graph, stream=side):
                 self.logits = self._body()
         torch.cuda.current_stream(dev).wait_stream(side)
-        kv_cache.cache_seqlens.copy_(saved_lens)
-        self._prev.copy_(self._prev_saved)
+        for t, value in zip(in_place, saved):
+            t.copy_(value)
 
     def _body(self):
-        if not hasattr(self, "_prev_saved"):
-            self._prev_saved = self._prev.clone()
-        self.cache.prev_embedding = self._prev
+        if self._prev is not None:
+            self.cache.prev_embedding = self._prev
         logits = self.model.forward(self.ids, kv_cache=self.cache)[:, -1, :]
-        self._prev.copy_(self.cache.prev_embedding)
-        self.cache.prev_embedding = self._prev
+        if self._prev is not None:
+            self._prev.copy_(self.cache.prev_embedding)
+            self.cache.prev_embedding = self._prev
         return logits
 
     def step(self, ids):

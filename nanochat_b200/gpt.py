@@ -10,7 +10,7 @@ sequence of torch ops as the reference, kept so that the path can be driven end 
 ``state_dict`` so its checkpoints load unchanged.  Training (loss, optimizers, autograd through
 attention) is out of scope and absent.
 """
-from dataclasses import dataclass
+from dataclasses import dataclass, fields
 
 import torch
 import torch.nn as nn
@@ -18,6 +18,7 @@ import torch.nn.functional as F
 
 from . import ops
 from .flash_attention import flash_attn
+from .models import register
 
 
 # ------------------------------------------------------------------------------------------------
@@ -208,6 +209,7 @@ class Block(nn.Module):
         return x + self.mlp(rms(x))
 
 
+@register("nanochat")
 class GPT(nn.Module):
     """Inference-only GPT with the reference's module tree and forward arithmetic (gpt.py:154-481)."""
 
@@ -240,6 +242,18 @@ class GPT(nn.Module):
         self.rotary_seq_len = config.sequence_len * 10  # same over-allocation as gpt.py:195
         self.register_buffer("cos", torch.empty(0), persistent=False)
         self.register_buffer("sin", torch.empty(0), persistent=False)
+
+    @classmethod
+    def from_dict(cls, config, tensors, dtype, device):
+        """From a model folder: config.json holds GPTConfig's fields, the tensors are the state_dict."""
+        names = {f.name for f in fields(GPTConfig)}
+        with torch.device("meta"):
+            model = cls(GPTConfig(**{k: v for k, v in config.items() if k in names}), compute_dtype=dtype)
+        model.load_state_dict({k: v.to(device=device, dtype=dtype) for k, v in tensors.items()}, assign=True)
+        for buffer in ("cos", "sin"):
+            setattr(model, buffer, torch.empty(0, device=device))
+        model.build_rotary()
+        return model.eval()
 
     def get_device(self):
         return self.transformer.wte.weight.device
