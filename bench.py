@@ -997,6 +997,210 @@ def run_case(args):
     print(json.dumps(out), flush=True)
 
 
+# ------------------------------------------------------------------------------------------------
+# Sipadra (wkv and parallel layers) beside the GPT of equal width and depth
+# ------------------------------------------------------------------------------------------------
+SIPADRA_SIZES = {
+    # GPT's relu^2 MLP holds 8 width^2 weights; ff is chosen so that the gated one holds about as many
+    "d24": dict(width=1536, n_layer=24, ff=4096, wkv_heads=24, left=(12, 12), window=1024, right=(12, 64, 128), rank=64),
+    "d32": dict(width=2048, n_layer=32, ff=5504, wkv_heads=32, left=(16, 4), window=2048, right=(16, 128, 128), rank=96),
+}
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12  # nominal fp32 pipe at the maximum clock
+
+
+def sipadra_config(width, n_layer, ff, wkv_heads, left, window, right, rank, vocab=32768):
+    wkv = {"type": "wkv", "mixer": {"heads": wkv_heads, "dim": 64}, "mlp": {"kind": "dense", "ff": ff}}
+    par = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff}, "mixer": {
+        "left": {"heads": left[0], "kv_heads": left[1], "dim": 128, "vdim": 128, "mask": {"size": window}, "scale": 128 ** -0.5,
+                 "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+        "right": {"heads": right[0], "dim": right[1], "vdim": right[2],
+                  "decay": [1 - 2.0 ** -(3 + 6 * i / right[0]) for i in range(right[0])]},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    return {"architecture": "Sipadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": [par if i % 3 == 2 else wkv for i in range(n_layer)]}
+
+
+def build_sipadra(name, dev):
+    from nanochat_b200.sipadra import Sipadra, tensor_shapes
+    size = SIPADRA_SIZES[name]
+    cfg = sipadra_config(**size)
+    gen = torch.Generator(device=dev).manual_seed(11)
+    tensors = {}
+    for key, shape in tensor_shapes(cfg, size["rank"]).items():
+        z = torch.randn(shape, generator=gen, device=dev)
+        tensors[key] = (1 + 0.1 * z if "norm" in key else z.sigmoid() if ".mu." in key else z - 2 if key.endswith("w0")
+                        else z if key == "embed" else z * shape[-1] ** -0.5)
+    return Sipadra.from_dict(cfg, tensors, torch.bfloat16, dev)
+
+
+def build_gpt_like(name, dev):
+    from nanochat_b200.gpt import GPT, GPTConfig
+    size = SIPADRA_SIZES[name]
+    cfg = GPTConfig(sequence_len=4 * size["window"], vocab_size=32768, n_layer=size["n_layer"], n_head=size["left"][0],
+                    n_kv_head=size["left"][1], n_embd=size["width"])
+    with torch.device("meta"):
+        model = GPT(cfg, compute_dtype=torch.bfloat16)
+    model.to_empty(device=dev)
+    model.init_weights()
+    model.to(torch.bfloat16)
+    model.window_sizes = [(size["window"] - 1, 0)] * size["n_layer"]
+    return model
+
+
+def _time_cold(fn, iters, flush, warmup=3):
+    """Median seconds of single calls, L2 flushed before each (the flush also hides the host's launch time)."""
+    times = []
+    for i in range(warmup + iters):
+        flush.zero_()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        if i >= warmup:
+            times.append(e0.elapsed_time(e1) * 1e-3)
+    return sorted(times)[len(times) // 2]
+
+
+def sipadra_models(dev, iters):
+    """Whole-model prefill and decode tokens/s of both designs."""
+    from nanochat_b200.engine import GraphedDecodeStep, new_cache
+    rows = []
+    for name in SIPADRA_SIZES:
+        for kind, build in (("sipadra", build_sipadra), ("gpt", build_gpt_like)):
+            model = build(name, dev)
+            for Bc, T in ((1, 2048), (1, 8192), (8, 2048)):
+                cache = new_cache(model, Bc, T, torch.bfloat16)
+                ids = torch.randint(0, 32768, (Bc, T), generator=torch.Generator().manual_seed(1)).to(dev)
+
+                def run(i):
+                    cache.reset()
+                    model.forward(ids, kv_cache=cache)
+
+                sec = _time_cuda(run, iters)
+                rows.append({"model": kind, "size": name, "phase": "prefill", "rows": Bc, "tokens": T, "ms": sec * 1e3,
+                             "tokens_per_s": Bc * T / sec})
+                del cache
+            for Bc, ctx in ((1, 1024), (64, 1024), (256, 1024)):
+                cache = new_cache(model, Bc, ctx + 64, torch.bfloat16)
+                ids = torch.randint(0, 32768, (Bc, 16), generator=torch.Generator().manual_seed(2)).to(dev)
+                model.forward(ids, kv_cache=cache)
+                cache.cache_seqlens.fill_(ctx)  # as if ctx tokens were there; what the rows hold does not matter here
+                step = GraphedDecodeStep(model, cache, ids[:, :1].contiguous())
+
+                def one(i):
+                    cache.cache_seqlens.fill_(ctx)
+                    step.step(ids[:, :1])
+
+                sec = _time_cuda(one, max(iters, 20))
+                rows.append({"model": kind, "size": name, "phase": "decode", "rows": Bc, "context": ctx, "ms": sec * 1e3,
+                             "tokens_per_s": Bc / sec})
+                del step, cache
+            del model
+            torch.cuda.empty_cache()
+    return rows
+
+
+def sipadra_kernels(dev, iters, peak, tflops):
+    """Kernels of the design, and the GPT path's like kernels on the same sizes, against their rooflines."""
+    from nanochat_b200 import mixer_ops as mo, ops
+    from nanochat_b200.gpt import precompute_rotary_embeddings
+    from nanochat_b200.mixers import rotary_table
+    bf, f32 = torch.bfloat16, torch.float32
+    gen = torch.Generator(device=dev).manual_seed(12)
+    rnd = lambda *shape, dtype=bf: torch.randn(*shape, generator=gen, device=dev).to(dtype)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows = []
+
+    def note(kernel, shape, fn, nbytes=0, flops=0, peak_flops=None):
+        sec = _time_cold(fn, iters, flush)
+        need = max(nbytes / (peak * 1e9), flops / (peak_flops * 1e12) if flops else 0)
+        rows.append({"kernel": kernel, "shape": shape, "us": sec * 1e6, "roofline_us": need * 1e6, "frac": need / sec,
+                     "bound": "bytes" if nbytes / (peak * 1e9) >= need else "flops"})
+
+    for name, size in SIPADRA_SIZES.items():
+        W, H, D = size["width"], size["wkv_heads"], 64
+        Hr, Dr, Er = size["right"]
+        Hq, Hkv = size["left"]
+        HD = H * D
+        norm_w, x0, u = rnd(HD, dtype=f32), rnd(HD, dtype=f32) - 2, rnd(HD, dtype=f32)
+        decay = torch.full((Hr,), 0.97, device=dev)
+        gw = rnd(Hr * Er, dtype=f32)
+        for Bc, T in ((1, 2048), (1, 8192), (8, 2048), (64, 1), (256, 1)):
+            N, shape = Bc * T, f"{name} B{Bc} T{T}"
+            r, k, v, g = (rnd(N, HD) for _ in range(4))
+            x = rnd(N, HD, dtype=f32) * 0.5
+            st = torch.zeros(Bc, H, D, D, device=dev)
+            note("recurrent wkv", shape, lambda: mo.recurrent(r, k, v, st, Bc, T, H, D, D, decay_logits=x, decay_bias=x0, bonus=u, gate=g,
+                 norm_weight=norm_w, eps=1e-6), N * HD * 14 + 8 * st.numel(), 6 * N * HD * D, FP32_TFLOPS)
+            z = rnd(N, 2 * Hr * Dr + 2 * Hr * Er)
+            rq, rk, rv, rg = z.split([Hr * Dr, Hr * Dr, Hr * Er, Hr * Er], 1)
+            st2 = torch.zeros(Bc, Hr, Dr, Er, device=dev)
+            note("recurrent decay", shape, lambda: mo.recurrent(rq, rk, rv, st2, Bc, T, Hr, Dr, Er, decay=decay, silu_inputs=True),
+                 N * (Hr * Dr * 4 + Hr * Er * 6) + 8 * st2.numel(), 6 * N * Hr * Dr * Er, FP32_TFLOPS)
+            o32 = rnd(N, Hr * Er, dtype=f32)
+            note("gated_norm", shape, lambda: mo.gated_norm(o32, rg, gw, Hr * Er, 1e-6), N * Hr * Er * 8)
+            xs, y, w = rnd(N, W, dtype=f32), rnd(N, W), rnd(W, dtype=f32)
+            mu, carry = rnd(5, W, dtype=f32), rnd(Bc, W, dtype=f32)
+            note("resid_norm", shape, lambda: mo.resid_norm(xs, y, w, 1e-6, bf, Bc, T, want_h=True), N * W * 12)
+            note("resid_norm + 5 mixes", shape, lambda: mo.resid_norm(xs, y, w, 1e-6, bf, Bc, T, mu=mu, carry=carry), N * W * 20)
+            note("gpt: glue_mix_norm", shape, lambda: ops.glue_mix_norm(y, add=y, x0=y, resid_lambda=1.0, x0_lambda=0.1), N * W * 10)
+            gu = rnd(N, 2 * size["ff"])
+            note("silu_mul", shape, lambda: mo.silu_mul(gu), N * size["ff"] * 6)
+            h4 = rnd(N, 4 * W)
+            note("gpt: glue_relu_sq", shape, lambda: ops.glue_relu_sq(h4), N * W * 16)
+            ctx = 1024 if T == 1 else 0
+            cap = ctx + T
+            kc, vc = rnd(Bc, cap, Hkv, 128), rnd(Bc, cap, Hkv, 128)
+            lens = torch.full((Bc,), cap - T, dtype=torch.int32, device=dev)
+            qkv = rnd(N, (Hq + 2 * Hkv) * 128)
+            lq, lk, lv = qkv.split([Hq * 128, Hkv * 128, Hkv * 128], 1)
+            table = rotary_table(cap, 128, 5e5, None, dev)
+            ab = N * (Hq + 2 * Hkv) * 512
+            note("rope_unit_append", shape, lambda: mo.rope_unit_append(lq, lk, lv, table, 128, kc, vc, lens, Bc, T, Hq, Hkv, 128, 128, 1.0, 1e-6),
+                 ab + cap * 512)
+            cos, sin = precompute_rotary_embeddings(cap, 128, device=dev)
+            q4, k4, v4 = (t.contiguous().view(Bc, T, -1, 128) for t in (lq, lk, lv))
+            note("gpt: append_rope_norm", shape, lambda: ops.append_rope_norm(q4, k4, v4, kc, vc, lens, cos, sin), ab + cap * 256)
+            win = size["window"]
+            if T == 1:
+                nb, fl = 4 * Bc * Hkv * 128 * min(win, cap) + 4 * N * Hq * 128, 0
+            else:
+                pairs = sum(min(i + 1, win) for i in range(T))
+                nb, fl = 4 * N * (Hq + Hkv) * 128, 512 * Bc * Hq * pairs
+            note("split_p attention", shape, lambda: mo.split_p_attention(q4, kc, vc, lens, win), nb, fl, tflops)
+            if T == 1:
+                note("gpt: decode_attention", shape, lambda: ops.decode_attention(q4[:, 0], kc, vc, lens, 1, win - 1), nb, fl, tflops)
+            else:
+                note("gpt: prefill_attention", shape, lambda: ops.prefill_attention(q4, kc, vc, lens, win - 1), nb, fl, tflops)
+            del r, k, v, g, x, st, z, o32, xs, y, gu, h4, kc, vc, qkv, q4, k4, v4
+    return rows
+
+
+def run_sipadra_case(args):
+    from nanochat_b200 import ops
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peak, kind = peaks()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tflops = float(json.load(f)["bf16_tflops"])
+    except Exception:
+        tflops = 1590.0
+    iters = min(max(args.steps, 5), 20)
+    out = {"case": args.case, "n_gpus": 1, "data": "synthetic", "dtype": "bf16", "peak_gbs": peak, "peak_tflops": tflops,
+           "peak_kind": f"of {kind}", "fp32_tflops_nominal": FP32_TFLOPS, "sizes": SIPADRA_SIZES, "iters": iters}
+    sampler = ClockSampler(0)
+    sampler.start()
+    with torch.no_grad():
+        if args.case == "sipadra":
+            out["models"] = sipadra_models(dev, iters)
+        out["kernels"] = sipadra_kernels(dev, iters, peak, tflops)
+    out["clocks"] = sampler.stop()
+    out["device_status"] = ops.read_status(dev)
+    print(json.dumps(out), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1011,11 +1215,13 @@ def main():
     ap.add_argument("--case", default=None,
                     help="secondary op-level measurement instead of the headline workload: decode_long, decode_gqa, "
                          "decode_gqa_window, decode_d24, decode_paged, prefill, prefill_paged, train_attn, broadcast, append, engine_d24, engine_d24_small, engine_d32, "
-                         "engine_d32_small, engine_api_d24, engine_api_small")
+                         "engine_d32_small, engine_api_d24, engine_api_small; sipadra (both models and kernels), sipadra_kernels")
     args = ap.parse_args()
     global REGIONS_OVERRIDE
     REGIONS_OVERRIDE = args.regions
-    if args.case:
+    if args.case in ("sipadra", "sipadra_kernels"):
+        run_sipadra_case(args)
+    elif args.case:
         run_case(args)
     elif args.impl == "reference":
         run_reference(args)

@@ -62,6 +62,23 @@ __device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[4]) {
     *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]));
 }
 
+__device__ __forceinline__ void get_v(const float *p, float (&o)[8]) {
+    const float4 a = reinterpret_cast<const float4 *>(p)[0], b = reinterpret_cast<const float4 *>(p)[1];
+    o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
+}
+__device__ __forceinline__ void get_v(const __nv_bfloat16 *p, float (&o)[8]) {
+    const uint4 f = *reinterpret_cast<const uint4 *>(p);
+    o[0] = bf16lo(f.x); o[1] = bf16hi(f.x); o[2] = bf16lo(f.y); o[3] = bf16hi(f.y);
+    o[4] = bf16lo(f.z); o[5] = bf16hi(f.z); o[6] = bf16lo(f.w); o[7] = bf16hi(f.w);
+}
+__device__ __forceinline__ void put_v(float *p, const float (&o)[8]) {
+    reinterpret_cast<float4 *>(p)[0] = make_float4(o[0], o[1], o[2], o[3]);
+    reinterpret_cast<float4 *>(p)[1] = make_float4(o[4], o[5], o[6], o[7]);
+}
+__device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[8]) {
+    *reinterpret_cast<uint4 *>(p) = make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
+}
+
 __device__ __forceinline__ float block_sum(float v, float *s_part) {
 #pragma unroll
     for (int off = 16; off; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
@@ -110,7 +127,7 @@ __global__ void __launch_bounds__(RN_THREADS) resid_norm_kernel(const ResidNormP
                 for (int e = 0; e < V; ++e) ss = fmaf(y[k][e], y[k][e], ss);
             }
         }
-        const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)p.W + p.eps);
+        const float inv = rsqrtf(block_sum(ss, s_part) / (float)p.W + p.eps);
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
             const int c = (k * RN_THREADS + tid) * V;
@@ -147,7 +164,7 @@ __global__ void __launch_bounds__(RN_THREADS) resid_norm_kernel(const ResidNormP
                     for (int e = 0; e < V; ++e) ss = fmaf(cur[k][e], cur[k][e], ss);
                 }
             }
-            inv_f = 1.f / sqrtf(block_sum(ss, s_part) / (float)p.W + p.eps);
+            inv_f = rsqrtf(block_sum(ss, s_part) / (float)p.W + p.eps);
         }
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
@@ -169,6 +186,7 @@ __global__ void __launch_bounds__(RN_THREADS) resid_norm_kernel(const ResidNormP
             }
             if (p.mix) {
                 const long long plane = (long long)p.B * p.T * p.W;
+#pragma unroll 5
                 for (int m = 0; m < p.n_mix; ++m) {
                     float mu[V], o[V];
                     get_v(p.mu + (long long)m * p.W + c, mu);
@@ -190,15 +208,19 @@ template <typename T>
 __global__ void __launch_bounds__(256) silu_mul_kernel(const T *__restrict__ in, T *__restrict__ out, long long rows, int F, int vec) {
     const long long step = (long long)gridDim.x * blockDim.x;
     if (vec) {
-        const long long per_row = F / 4, n = rows * per_row;
-        for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += step) {
-            const long long row = i / per_row;
-            const int c = (int)(i - row * per_row) * 4;
-            float g[4], u[4], o[4];
+        // 8 channels at a time, a row per CTA turn
+        const int per_row = F / 8, blocks_per_row = (per_row + 255) / 256;
+        const long long n = rows * blocks_per_row;
+        for (long long i = blockIdx.x; i < n; i += gridDim.x) {
+            const long long row = i / blocks_per_row;
+            const int c = ((int)(i - row * blocks_per_row) * 256 + threadIdx.x) * 8;
+            if (c >= F) continue;
+            float g[8], u[8], o[8];
             get_v(in + row * 2 * F + c, g);
             get_v(in + row * 2 * F + F + c, u);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) o[e] = g[e] / (1.f + expf(-g[e])) * u[e];
+            for (int e = 0; e < 8; ++e)
+                o[e] = (sizeof(T) == 2 ? __fdividef(g[e], 1.f + __expf(-g[e])) : g[e] / (1.f + expf(-g[e]))) * u[e];
             put_v(out + row * F + c, o);
         }
     } else {
@@ -231,8 +253,15 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float *__restrict
 }
 
 __global__ void __launch_bounds__(256) softcap_kernel(float *z, long long n, float cap) {
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
-        z[i] = cap * tanhf(z[i] / cap);
+    const long long step = (long long)gridDim.x * blockDim.x, first = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const long long quads = (((uintptr_t)z) & 15) == 0 ? n / 4 : 0;
+    for (long long i = first; i < quads; i += step) {
+        float4 f = reinterpret_cast<float4 *>(z)[i];
+        f.x = cap * tanhf(f.x / cap); f.y = cap * tanhf(f.y / cap);
+        f.z = cap * tanhf(f.z / cap); f.w = cap * tanhf(f.w / cap);
+        reinterpret_cast<float4 *>(z)[i] = f;
+    }
+    for (long long i = quads * 4 + first; i < n; i += step) z[i] = cap * tanhf(z[i] / cap);
 }
 
 static unsigned grid_for(long long n) {
@@ -307,10 +336,9 @@ int nckv_silu_mul(const void *gate_up, void *out, int64_t rows, int F, int f32, 
         set_error("silu_mul: null pointer or non-positive size");
         return NCKV_E_ARG;
     }
-    const uintptr_t elem = f32 ? 4 : 2;
-    const int vec = F % 4 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & (4 * elem - 1)) == 0;
+    const int vec = F % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const unsigned grid = grid_for(rows * (vec ? F / 4 : F));
+    const unsigned grid = vec ? grid_for(rows * ((F / 8 + 255) / 256) * 256) : grid_for(rows * F);
     if (f32) silu_mul_kernel<float><<<grid, 256, 0, s>>>(static_cast<const float *>(gate_up), static_cast<float *>(out), rows, F, vec);
     else silu_mul_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(static_cast<const __nv_bfloat16 *>(gate_up), static_cast<__nv_bfloat16 *>(out), rows, F, vec);
     NCKV_CUDA_CHECK(cudaGetLastError());
@@ -334,7 +362,7 @@ int nckv_softcap(float *z, int64_t n, float cap, void *stream) {
         set_error("softcap: null pointer, non-positive size or cap");
         return NCKV_E_ARG;
     }
-    softcap_kernel<<<grid_for(n), 256, 0, static_cast<cudaStream_t>(stream)>>>(z, n, cap);
+    softcap_kernel<<<grid_for((n + 3) / 4), 256, 0, static_cast<cudaStream_t>(stream)>>>(z, n, cap);
     NCKV_CUDA_CHECK(cudaGetLastError());
     return NCKV_OK;
 }

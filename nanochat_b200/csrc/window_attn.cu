@@ -99,7 +99,7 @@ __global__ void __launch_bounds__(256) rope_unit_append_kernel(const RopeUnitPar
         if (!is_v) {
 #pragma unroll
             for (int off = 16; off; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-            f = 1.f / sqrtf(ss / (float)D + p.eps);
+            f = rsqrtf(ss / (float)D + p.eps);
             if (is_q) f *= p.q_scale;
         }
 #pragma unroll

@@ -41,6 +41,33 @@ class SipadraConfig:
         return cls(c["vocab"], c["width"], c["norm"]["eps"], c.get("logit_softcap"), c["layers"])
 
 
+def tensor_shapes(config, rank):
+    """name -> shape of every tensor of a configuration (a dict as in config.json); ``rank`` is the inner width
+    of the decay paths, which the configuration leaves to the tensors."""
+    W = config["width"]
+    shapes = {"embed": (config["vocab"], W), "final.norm": (W,)}
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}."
+        shapes[p + "norm1"] = (W,)
+        if layer["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            shapes.update({f"{p}mix.mu.{s}": (W,) for s in WkvMixer.MIXES})
+            shapes.update({f"{p}mix.{s}": (n, W) for s in "rkvg"})
+            shapes.update({p + "mix.w1": (rank, W), p + "mix.w2": (n, rank), p + "mix.w0": (n,),
+                           p + "mix.u": (m["heads"], m["dim"]), p + "mix.norm": (n,), p + "mix.o": (W, n)})
+        else:
+            a, b, left, right = m["left"], m["right"], p + "mix.left.", p + "mix.right."
+            out, n = a["heads"] * a["vdim"], b["heads"] * b["vdim"]
+            shapes.update({left + "q": (a["heads"] * a["dim"], W), left + "k": (a["kv_heads"] * a["dim"], W),
+                           left + "v": (a["kv_heads"] * a["vdim"], W), left + "o": (W, out),
+                           right + "q": (b["heads"] * b["dim"], W), right + "k": (b["heads"] * b["dim"], W),
+                           right + "v": (n, W), right + "g": (n, W), right + "norm": (n,), right + "o": (W, n)})
+        if layer.get("mlp") is not None:
+            ff = layer["mlp"]["ff"]
+            shapes.update({p + "norm2": (W,), p + "mlp.gate": (ff, W), p + "mlp.up": (ff, W), p + "mlp.down": (W, ff)})
+    return shapes
+
+
 class _Scope:
     """The tensors below a name prefix, looked up without it."""
 
@@ -101,6 +128,12 @@ class Sipadra:
 
     @classmethod
     def from_dict(cls, config, tensors, dtype, device):
+        for name, shape in tensor_shapes(config, rank=None).items():
+            if name not in tensors:
+                raise ValueError(f"the weights lack {name}")
+            have = tuple(tensors[name].shape)
+            if len(have) != len(shape) or any(want not in (None, n) for want, n in zip(shape, have)):
+                raise ValueError(f"{name} is {have}, the configuration says {shape}")
         tensors = {k: v.to(device=device, dtype=dtype) for k, v in tensors.items()}
         return cls(SipadraConfig.from_dict(config), tensors, dtype)
 
