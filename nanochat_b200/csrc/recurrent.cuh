@@ -15,15 +15,19 @@
 // Mapping.  A CTA owns up to 128 value columns of one (row, head, segment).  A warp owns VG*8 of them:
 // lane = vg * KG + kg holds key channels {4 KG i + 4 kg + j : i < U, j < 4} of columns {8 vg + c : c < 8}.
 // Pairs of key channels are the two halves of packed fp32 instructions; a step is three of them per
-// pair and column.  Tokens run in batches of TB = 4: their partial outputs are summed over the KG lanes
+// pair and column.  Tokens run in batches of 4: their partial outputs are summed over the KG lanes
 // together (a reduce-scatter that leaves a lane 2 or 4 columns of one token), so the latency of the
 // shuffles is paid once per batch.  Batches are padded with tokens that leave the state as it is
 // (k = 0, w = 1).  Per warp and token 3 U + 2 16-byte shared-memory loads stand against 48 U packed
 // multiply-adds: the fp32 pipe is the bound, shared memory and the issue slots are just below it.  Tokens are staged C at a time through two buffers
 // (converted, activated and exponentiated once per head on the way, by all warps evenly); the next
 // chunk's bytes wait in registers meanwhile.  8 threads normalise, gate and store a token of the
-// chunk before.  A single-token call (TB = 1) is the same code with one chunk of one: 16-byte state loads
-// and stores that are all in flight together, which is what a decode step is bound by.
+// chunk before.
+//
+// Single tokens.  recurrent_step_kernel: a decode step is bound by reading and writing the state, so it
+// runs more and smaller threads: a thread owns 4 value columns of every (256 / column quads)-th or so key
+// row, a row of the state is one coalesced run, and 8 rows per thread are in flight before the first
+// is needed.
 //
 // Segments.  Few (row, head) pairs and a long prompt leave most SMs idle.  Then the prompt is cut
 // into segments that run side by side: a first pass finds each segment's own contribution to the
@@ -60,6 +64,7 @@ struct RecurrentParams {
 };
 
 constexpr int REC_COLS = 128;  // value columns per CTA
+constexpr int REC_BATCH = 4;   // tokens whose outputs are reduced together
 constexpr int REC_MAXQ = 2;    // 4-element pieces a thread stages per vector and chunk
 
 // fp32 activations get the full-precision functions, bf16 ones the fast intrinsics (a few fp32 ulps)
@@ -162,9 +167,9 @@ template <int BIT, int LEN> __device__ __forceinline__ int reduce_scatter(float 
 }
 
 // CHANNEL: decay per token and key channel, bonus form.  OUT: false in the first pass over segments.
-template <typename T, int KG, int U, int TB, bool CHANNEL, bool OUT, bool VEC>
+template <typename T, int KG, int U, bool CHANNEL, bool OUT, bool VEC>
 __global__ void __launch_bounds__(REC_COLS / (256 / KG) * 32) recurrent_kernel(const RecurrentParams p) {
-    constexpr int VG = 32 / KG, KP = 4 * KG * U, KQ = KP / 4, WC = 8 * VG;  // WC: columns per warp
+    constexpr int TB = REC_BATCH, VG = 32 / KG, KP = 4 * KG * U, KQ = KP / 4, WC = 8 * VG;  // WC: columns per warp
     constexpr int NB = KQ > 32 ? KQ / 32 : 1;                               // partial bonus sums per token
     const int NT = blockDim.x, NW = NT >> 5;
     const int VP = NW * WC, VQ = VP / 4;
@@ -287,7 +292,7 @@ __global__ void __launch_bounds__(REC_COLS / (256 / KG) * 32) recurrent_kernel(c
         const int n = min(C, t_end - t0);
         const float *buf = s_buf + parity * per_buf;
         float *so = s_out + parity * C * VP;
-        const bool more = TB > 1 && t0 + C < t_end;  // TB 1: single-token calls
+        const bool more = t0 + C < t_end;
         if (more) fetch(t0 + C);
         Quad<T> rg[REC_COLS / 32];
         if (gated) {  // the gate of this chunk, needed at its end (later tokens of a short CTA's share: loaded there)
@@ -320,7 +325,7 @@ __global__ void __launch_bounds__(REC_COLS / (256 / KG) * 32) recurrent_kernel(c
                         w2[2 * i] = make_float2(f.x, f.y);
                         w2[2 * i + 1] = make_float2(f.z, f.w);
                     } else {
-                        const float wt = TB == 1 || t < n ? w_head : 1.f;
+                        const float wt = t < n ? w_head : 1.f;
                         w2[2 * i] = w2[2 * i + 1] = make_float2(wt, wt);
                     }
                 }
@@ -348,19 +353,17 @@ __global__ void __launch_bounds__(REC_COLS / (256 / KG) * 32) recurrent_kernel(c
             }
             if (OUT) {
                 const int first = reduce_scatter<KG / 2, TB * 8>(o, kg);
-                constexpr int HELD = TB * 8 >= KG ? TB * 8 / KG : 1;  // 4, 2 or 1 columns of one token
+                constexpr int HELD = TB * 8 / KG;  // 4 or 2 columns of one token
                 const int t = tb + first / 8, col = v0 + first % 8;
-                if (HELD * KG == TB * 8 || (kg & 1) == 0) {
-                    float bonus = 0.f;
-                    if (CHANNEL) {
-                        bonus = buf[off_b + t * 4];
-                        if (NB > 1) bonus += buf[off_b + t * 4 + 1];
-                    }
+                float bonus = 0.f;
+                if (CHANNEL) {
+                    bonus = buf[off_b + t * 4];
+                    if (NB > 1) bonus += buf[off_b + t * 4 + 1];
+                }
 #pragma unroll
-                    for (int c = 0; c < HELD; ++c) {
-                        if (CHANNEL) o[c] = fmaf(bonus, buf[off_v + t * VP + col + c], o[c]);
-                        so[t * VP + col + c] = o[c];
-                    }
+                for (int c = 0; c < HELD; ++c) {
+                    if (CHANNEL) o[c] = fmaf(bonus, buf[off_v + t * VP + col + c], o[c]);
+                    so[t * VP + col + c] = o[c];
                 }
             }
         }
@@ -432,9 +435,127 @@ __global__ void __launch_bounds__(REC_COLS / (256 / KG) * 32) recurrent_kernel(c
     }
 }
 
-template <typename T, int KG, int U, int TB, bool CHANNEL, bool OUT, bool VEC>
+// One token per row.  Thread = row group * CQ + column quad; CQ (a power of two) quads cover the CTA's columns.
+template <typename T, bool CHANNEL>
+__global__ void __launch_bounds__(256) recurrent_step_kernel(const RecurrentParams p, int CQ) {
+    constexpr int ROWS = 8;  // state rows a thread has in flight
+    extern __shared__ __align__(16) float step_smem[];
+    float4 *s_kqw = reinterpret_cast<float4 *>(step_smem);       // (Dk): k, q, w
+    float4 *s_red = s_kqw + p.Dk;                                 // (warps, CQ) partial outputs
+    __shared__ float s_bonus[8];
+    const int NT = blockDim.x, RG = NT / CQ, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int h = blockIdx.x / p.n_cols, b = blockIdx.y, col0 = (blockIdx.x % p.n_cols) * CQ * 4;
+    const int Dk = p.Dk, cq = tid % CQ, rg = tid / CQ, col = col0 + cq * 4;
+    const bool have_col = col < p.Dv;
+    const long long base = ((long long)b * p.H + h) * Dk * p.Dv + col;
+    const float *src = p.state_in + base;
+    float *dst = p.state_out + base;
+
+    float4 S[ROWS];
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const int r = rg + i * RG;
+        S[i] = load_quad<true>(src + (long long)r * p.Dv, have_col && r < Dk, 4).w;
+    }
+    const float4 v_raw = widen(load_quad<true>(static_cast<const T *>(p.v) + b * p.v_stride + (long long)h * p.Dv + col, have_col, 4));
+    const bool gated = CHANNEL && p.norm_w != nullptr, last = tid < CQ && have_col;
+    const Quad<T> gate = load_quad<true>(static_cast<const T *>(p.gate) + b * p.gate_stride + (long long)h * p.Dv + col, gated && last, 4);
+    const float4 nw = load_quad<true>(p.norm_w + (long long)h * p.Dv + col, gated && last, 4).w;
+    float bonus = 0.f;
+    const float w_head = CHANNEL ? 0.f : p.decay[h];
+    for (int c = tid; c < Dk; c += NT) {
+        auto one = [](const T *ptr) {
+            if constexpr (sizeof(T) == 2) return bf16_bits_to_float(*reinterpret_cast<const uint16_t *>(ptr));
+            else return *ptr;
+        };
+        float q = one(static_cast<const T *>(p.q) + b * p.q_stride + (long long)h * Dk + c);
+        float k = one(static_cast<const T *>(p.k) + b * p.k_stride + (long long)h * Dk + c);
+        if (p.act_in) {
+            q = silu_of<T>(q);
+            k = silu_of<T>(k);
+        }
+        float w = w_head;
+        if (CHANNEL) {
+            w = exp_of<T>(-exp_of<T>(p.x[b * p.x_stride + (long long)h * Dk + c] + p.x0[h * Dk + c]));
+            bonus = fmaf(q * p.u[h * Dk + c], k, bonus);
+        }
+        s_kqw[c] = make_float4(k, q, w, 0.f);
+    }
+    const float4 v4 = p.act_in ? silu4<T>(v_raw) : v_raw;
+    if (CHANNEL) {
+#pragma unroll
+        for (int off = 16; off; off >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, off);
+        if (lane == 0) s_bonus[warp] = bonus;
+    }
+    __syncthreads();
+
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int r0 = 0; r0 < Dk; r0 += ROWS * RG) {
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            const int r = r0 + rg + i * RG;
+            if (r0 > 0) S[i] = load_quad<true>(src + (long long)r * p.Dv, have_col && r < Dk, 4).w;
+        }
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            const int r = r0 + rg + i * RG;
+            if (r >= Dk) continue;
+            const float4 f = s_kqw[r];
+            float4 n;
+            n.x = fmaf(f.z, S[i].x, f.x * v4.x); n.y = fmaf(f.z, S[i].y, f.x * v4.y);
+            n.z = fmaf(f.z, S[i].z, f.x * v4.z); n.w = fmaf(f.z, S[i].w, f.x * v4.w);
+            const float4 o = CHANNEL ? S[i] : n;
+            acc.x = fmaf(f.y, o.x, acc.x); acc.y = fmaf(f.y, o.y, acc.y);
+            acc.z = fmaf(f.y, o.z, acc.z); acc.w = fmaf(f.y, o.w, acc.w);
+            if (have_col) *reinterpret_cast<float4 *>(dst + (long long)r * p.Dv) = n;
+        }
+    }
+    for (int off = 16; off >= CQ; off >>= 1) {
+        acc.x += __shfl_xor_sync(0xffffffffu, acc.x, off); acc.y += __shfl_xor_sync(0xffffffffu, acc.y, off);
+        acc.z += __shfl_xor_sync(0xffffffffu, acc.z, off); acc.w += __shfl_xor_sync(0xffffffffu, acc.w, off);
+    }
+    if (lane < CQ) s_red[warp * CQ + lane] = acc;
+    __syncthreads();
+    if (warp > 0) return;  // CQ <= 32: the first warp finishes
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (last) {
+        float bn = 0.f;
+        for (int i = 0; i < (NT >> 5); ++i) {
+            const float4 f = s_red[i * CQ + cq];
+            o.x += f.x; o.y += f.y; o.z += f.z; o.w += f.w;
+            if (CHANNEL) bn += s_bonus[i];
+        }
+        o.x = fmaf(bn, v4.x, o.x); o.y = fmaf(bn, v4.y, o.y); o.z = fmaf(bn, v4.z, o.z); o.w = fmaf(bn, v4.w, o.w);
+    }
+    if (gated) {
+        float ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, o.w * o.w)));
+#pragma unroll
+        for (int off = 16; off; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        const float inv = rsqrtf(ss / (float)p.Dv + p.eps);
+        const float4 g = silu4<T>(widen(gate));
+        if (last)
+            store_quad<true>(static_cast<T *>(p.out) + b * p.out_stride + (long long)h * p.Dv + col,
+                             make_float4(o.x * inv * nw.x * g.x, o.y * inv * nw.y * g.y, o.z * inv * nw.z * g.z, o.w * inv * nw.w * g.w), 4);
+    } else if (last) {
+        store_quad<true>(static_cast<float *>(p.out) + b * p.out_stride + (long long)h * p.Dv + col, o, 4);
+    }
+}
+
+template <typename T, bool CHANNEL>
+static cudaError_t rec_step_launch(RecurrentParams p, cudaStream_t s) {
+    const int cols = p.Dv < REC_COLS ? p.Dv : REC_COLS;
+    int CQ = 1;
+    while (CQ * 4 < cols) CQ *= 2;
+    p.n_cols = (p.Dv + CQ * 4 - 1) / (CQ * 4);
+    const int NT = p.Dk * CQ > 1024 ? 256 : (p.Dk * CQ > 512 ? 128 : 64);  // about 8 rows of the state per thread
+    const size_t smem = sizeof(float4) * (p.Dk + (size_t)(NT / 32) * CQ);
+    recurrent_step_kernel<T, CHANNEL><<<dim3(p.H * p.n_cols, p.B), NT, smem, s>>>(p, CQ);
+    return cudaGetLastError();
+}
+
+template <typename T, int KG, int U, bool CHANNEL, bool OUT, bool VEC>
 static cudaError_t rec_launch_one(RecurrentParams p, cudaStream_t s) {
-    constexpr int WC = 256 / KG, KP = 4 * KG * U;
+    constexpr int TB = REC_BATCH, WC = 256 / KG, KP = 4 * KG * U;
     const int cols = p.Dv < REC_COLS ? p.Dv : REC_COLS;
     int NW = (cols + WC - 1) / WC;
     while (REC_MAXQ * NW * 32 < TB * (KP / 4)) ++NW;  // room to stage a batch (wide keys, few value columns)
@@ -443,37 +564,30 @@ static cudaError_t rec_launch_one(RecurrentParams p, cudaStream_t s) {
     const int Cv = REC_MAXQ * (NT / (VP / 4));
     if (Cv < C) C = Cv;
     if (C > 16) C = 16;
-    p.C = C = TB == 1 ? 1 : C - C % TB;
+    p.C = C -= C % TB;
     p.n_cols = (p.Dv + VP - 1) / VP;
     const size_t smem = sizeof(float) * (2ull * KP + VP + 2ull * C * (KP + VP + (OUT ? KP : 0) + (CHANNEL ? KP : 0) + (OUT && CHANNEL ? 4 : 0)) +
                                          (OUT ? 2ull * C * VP : 0));
     if (smem > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(recurrent_kernel<T, KG, U, TB, CHANNEL, OUT, VEC>,
+        const cudaError_t e = cudaFuncSetAttribute(recurrent_kernel<T, KG, U, CHANNEL, OUT, VEC>,
                                                    cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
-    recurrent_kernel<T, KG, U, TB, CHANNEL, OUT, VEC><<<dim3(p.H * p.n_cols, p.B, p.n_seg), NT, smem, s>>>(p);
+    recurrent_kernel<T, KG, U, CHANNEL, OUT, VEC><<<dim3(p.H * p.n_cols, p.B, p.n_seg), NT, smem, s>>>(p);
     return cudaGetLastError();
 }
 
 template <typename T, bool CHANNEL, bool OUT, bool VEC>
 static cudaError_t rec_launch_dims(const RecurrentParams &p, cudaStream_t s) {
-    if constexpr (OUT) {
-        if (p.T == 1) {
-            if (p.Dk <= 32) return rec_launch_one<T, 8, 1, 1, CHANNEL, OUT, VEC>(p, s);
-            if (p.Dk <= 64) return rec_launch_one<T, 16, 1, 1, CHANNEL, OUT, VEC>(p, s);
-            if (p.Dk <= 128) return rec_launch_one<T, 16, 2, 1, CHANNEL, OUT, VEC>(p, s);
-            return rec_launch_one<T, 16, 4, 1, CHANNEL, OUT, VEC>(p, s);
-        }
-    }
-    if (p.Dk <= 32) return rec_launch_one<T, 8, 1, 4, CHANNEL, OUT, VEC>(p, s);
-    if (p.Dk <= 64) return rec_launch_one<T, 16, 1, 4, CHANNEL, OUT, VEC>(p, s);
-    if (p.Dk <= 128) return rec_launch_one<T, 16, 2, 4, CHANNEL, OUT, VEC>(p, s);
-    return rec_launch_one<T, 16, 4, 4, CHANNEL, OUT, VEC>(p, s);
+    if (p.Dk <= 32) return rec_launch_one<T, 8, 1, CHANNEL, OUT, VEC>(p, s);
+    if (p.Dk <= 64) return rec_launch_one<T, 16, 1, CHANNEL, OUT, VEC>(p, s);
+    if (p.Dk <= 128) return rec_launch_one<T, 16, 2, CHANNEL, OUT, VEC>(p, s);
+    return rec_launch_one<T, 16, 4, CHANNEL, OUT, VEC>(p, s);
 }
 
 template <typename T>
 static cudaError_t rec_launch(const RecurrentParams &p, bool with_out, cudaStream_t s) {
+    if (p.T == 1 && p.vec && with_out) return p.x ? rec_step_launch<T, true>(p, s) : rec_step_launch<T, false>(p, s);
     if (p.vec) {
         if (p.x) return with_out ? rec_launch_dims<T, true, true, true>(p, s) : rec_launch_dims<T, true, false, true>(p, s);
         return with_out ? rec_launch_dims<T, false, true, true>(p, s) : rec_launch_dims<T, false, false, true>(p, s);

@@ -266,6 +266,18 @@ class HybridCache:
             t.copy_(other.state[key].expand_as(t))
         self.cache_seqlens.fill_(p)
 
+    def load_row(self, row, other):
+        """Put a batch-1 sequence of any length into one row, so that unequal sequences decode as one batch."""
+        assert other.batch_size == 1 and self.kv.keys() == other.kv.keys() and self.state.keys() == other.state.keys()
+        p = other.get_pos()
+        assert p <= self.max_seq_len, f"a sequence of {p} tokens does not fit rows of {self.max_seq_len}"
+        for key, pair in self.kv.items():
+            for mine, theirs in zip(pair, other.kv[key]):
+                mine[row, :p].copy_(theirs[0, :p])
+        for key, t in self.state.items():
+            t[row].copy_(other.state[key][0])
+        self.cache_seqlens[row] = p
+
 
 class SequenceRunner:
     """Runs portions of live sequences through a model, one entry at a time, each from what its earlier

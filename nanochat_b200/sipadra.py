@@ -128,6 +128,7 @@ class Sipadra:
 
     @classmethod
     def from_dict(cls, config, tensors, dtype, device):
+        parsed = SipadraConfig.from_dict(config)
         for name, shape in tensor_shapes(config, rank=None).items():
             if name not in tensors:
                 raise ValueError(f"the weights lack {name}")
@@ -135,7 +136,7 @@ class Sipadra:
             if len(have) != len(shape) or any(want not in (None, n) for want, n in zip(shape, have)):
                 raise ValueError(f"{name} is {have}, the configuration says {shape}")
         tensors = {k: v.to(device=device, dtype=dtype) for k, v in tensors.items()}
-        return cls(SipadraConfig.from_dict(config), tensors, dtype)
+        return cls(parsed, tensors, dtype)
 
     def get_device(self):
         return self.embed.device
