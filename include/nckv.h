@@ -397,13 +397,18 @@ NCKV_API int nckv_glue_ve_gate(const void *v, int64_t v_row_stride, const void *
  * recurrent states and the residual stream are fp32 in both.
  *
  * nckv_prefill_attn_split_p, nckv_decode_attn_split_p: nckv_prefill_attn / nckv_decode_attn with every
- *   probability entering the product with V as two bf16 terms (16 bits of it).
+ *   probability entering the product with V as two bf16 terms (16 bits of it).  sink: every softmax has one
+ *   more term of score 0 without a value.  gate (may be null): every head's output is multiplied by the sigmoid
+ *   of its logit, rows of Hq logits, gate_stride elements apart.
  * nckv_rope_unit_append: rotates the first rot_dims channels of q and k (pairs i, i + rot_dims / 2; cos_sin is
  *   (rope_len, rot_dims) fp32, cosines then sines, any amplitude included), divides q and k by their root mean
  *   square over Dk, multiplies q by q_scale; q -> q_out (B, T, Hq, Dk_pad), k and v -> the caches (token stride,
  *   then heads of Dk_pad / Dv_pad channels) at cache_seqlens[b] + t.  Padding is written as zeros.  q, k, v are
  *   rows of packed heads with their own row strides.
- * nckv_window_attn: query at position p sees keys j with 0 <= p - j < window; any head size up to 512, fp32 math.
+ * nckv_rms_rope_append: the same with one rms-norm over all of q's (and of k's) channels and weights, ahead of
+ *   the rotation.  k null: queries only, nothing is appended.
+ * nckv_window_attn: query at position p sees keys j with 0 <= p - j < window; any head size up to 512, fp32 math;
+ *   sink and gate as above.
  * nckv_recurrent: S <- diag(w) S + k v^T per head, state (B, H, Dk, Dv) fp32 read and updated in place.  With
  *   `x` (rows of H * Dk fp32): w = exp(-exp(x + x0)) per token and channel and o = (S_prev + diag(u) k v^T)^T q;
  *   else w = decay[h] and o = S^T q.  act_in: silu on q, k and v.  With norm_w: out = o / rms(o) * norm_w * silu(gate)
@@ -415,14 +420,30 @@ NCKV_API int nckv_glue_ve_gate(const void *v, int64_t v_row_stride, const void *
  *   updated).  x_out must not alias x when mix is given.
  * nckv_silu_mul: rows [gate | up] of 2F -> silu(gate) * up.  nckv_tanh_split: tanh(z), fp32 or bf16 [hi | lo].
  * nckv_softcap: z = cap * tanh(z / cap) in place.
+ * nckv_hyper_norm: S residual streams (rows, S, W): x_t' = sum_s mix[s, t] x_s + out[t] * (sum of the `parts`
+ *   rows of y), or table[token] in all of them; h = layer norm (mean taken off, weight, no bias) of
+ *   sum_t in[t] x_t' (in null: the plain sum).  x_out may be x, or null.  S <= 8.
+ * nckv_short_conv: causal convolution of up to 16 taps per channel, taps (K, C) with the current token's last;
+ *   out = act(bias + sum taps * (x + in_bias)), act: silu.  carry (B, K - 1, C) holds the inputs before the call.
+ * nckv_gated_scan: a = exp(-rate * sigmoid(r)); S = a S + sqrt(1 - a^2) sigmoid(i) u; out = S * gelu_tanh(y + y_bias).
+ *   gates (blocks, B * T, 2 C / blocks) holds the logits of r, then of i, without gate_bias (2, C).
+ * nckv_delta_rule, nckv_delta_step: S <- diag(exp(-rate softplus(x + x0))) S; u = sigmoid(b) (v - S^T k);
+ *   S <- S + k u^T; o = S^T q with q, k divided by sqrt(sum of squares + 1e-6) and q by sqrt(Dk).  H heads, G of
+ *   them for q and k.  The rule leaves o as (B * T, H * Dv) fp32 (Dk <= 256); the step takes one token per row
+ *   and leaves o / rms(o) * norm_w * sigmoid(gate) (Dv <= 128).
+ * nckv_route: per row the `top` largest of E logits; (row, choice) pairs sorted by expert: slot[i] = row * top +
+ *   choice, scale[i] = sigmoid(logit), expert e at [offsets[e], offsets[e + 1]).
+ * nckv_experts: up: out[i] = silu(s g) * (s u), [g; u] = w[e] a[slot[i] / top], s = scale[i], w (E, 2 N, K);
+ *   else out[slot[i]] = w[e] a[i], w (E, N, K).  R = rows * top pairs.
  */
 NCKV_API int nckv_prefill_attn_split_p(const void *q, const void *k, const void *v, const int32_t *cache_seqlens, void *out,
                       int B, int T_new, int Hq, int Hkv, int D, int T_k, int64_t kv_batch_stride,
-                      int64_t kv_token_stride, int window_left, int32_t *status, void *stream);
+                      int64_t kv_token_stride, int window_left, int sink, const void *gate, int64_t gate_stride,
+                      int32_t *status, void *stream);
 NCKV_API int nckv_decode_attn_split_p(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens,
                       void *out, int B, int Hq, int Hkv, int D, int T_max, int64_t cache_batch_stride,
-                      int64_t cache_token_stride, int seqlen_offset, int window_left, void *workspace,
-                      size_t workspace_bytes, void *stream);
+                      int64_t cache_token_stride, int seqlen_offset, int window_left, int sink, const void *gate,
+                      int64_t gate_stride, void *workspace, size_t workspace_bytes, void *stream);
 NCKV_API int nckv_rope_unit_append(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                       const float *cos_sin, const int32_t *cache_seqlens, void *q_out, void *k_cache, void *v_cache,
                       int64_t k_batch_stride, int64_t k_token_stride, int64_t v_batch_stride, int64_t v_token_stride,
@@ -430,7 +451,8 @@ NCKV_API int nckv_rope_unit_append(const void *q, const void *k, const void *v, 
                       int T_max, float q_scale, float eps, int f32, int32_t *status, void *stream);
 NCKV_API int nckv_window_attn(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens, void *out,
                       int64_t k_batch_stride, int64_t k_token_stride, int64_t v_batch_stride, int64_t v_token_stride, int B,
-                      int T, int Hq, int Hkv, int Dk, int Dv, int T_max, int window, float scale, int f32, void *stream);
+                      int T, int Hq, int Hkv, int Dk, int Dv, int T_max, int window, float scale, int sink, const void *gate,
+                      int64_t gate_stride, int f32, void *stream);
 NCKV_API size_t nckv_recurrent_workspace_bytes(int B, int T, int H, int Dk, int Dv);
 NCKV_API int nckv_recurrent(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                       const float *x, int64_t x_stride, const float *x0, const float *u, const float *decay,
@@ -445,6 +467,34 @@ NCKV_API int nckv_resid_norm(const float *x, const void *y, int y_f32, const flo
 NCKV_API int nckv_silu_mul(const void *gate_up, void *out, int64_t rows, int F, int f32, void *stream);
 NCKV_API int nckv_tanh_split(const float *z, void *out, int64_t rows, int R, int f32, void *stream);
 NCKV_API int nckv_softcap(float *z, int64_t n, float cap, void *stream);
+NCKV_API int nckv_rms_rope_append(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *q_weight, const float *k_weight, const float *cos_sin, const int32_t *cache_seqlens,
+                      void *q_out, void *k_cache, void *v_cache, int64_t k_batch_stride, int64_t k_token_stride,
+                      int64_t v_batch_stride, int64_t v_token_stride, int B, int T, int Hq, int Hkv, int Dk, int Dv,
+                      int Dk_pad, int Dv_pad, int rot_dims, int rope_len, int T_max, float q_scale, float eps, int f32,
+                      int32_t *status, void *stream);
+NCKV_API int nckv_hyper_norm(const float *x, const int64_t *tokens, const void *table, int vocab, const void *y, int parts,
+                      const float *mix, const float *out, const float *in, const float *w, float *x_out, void *h, int rows,
+                      int S, int W, float eps, int f32, void *stream);
+NCKV_API int nckv_short_conv(const void *x, int64_t x_stride, const float *taps, const float *in_bias, const float *bias, float *carry,
+                      void *out, int B, int T, int C, int K, int act, int f32, void *stream);
+NCKV_API int nckv_gated_scan(const void *u, int64_t u_stride, const void *y, int64_t y_stride, const float *gates,
+                      const float *gate_bias, const float *y_bias, const float *rate, float *state, void *out, int B, int T,
+                      int C, int blocks, int f32, void *stream);
+NCKV_API size_t nckv_delta_workspace_bytes(int B, int T, int H, int Dk);
+NCKV_API int nckv_delta_rule(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *x, int64_t x_stride, const float *x0, const float *rate, const void *b, int64_t b_stride,
+                      float *out, float *state, int B, int T, int H, int G, int Dk, int Dv, int f32, void *workspace,
+                      size_t workspace_bytes, void *stream);
+NCKV_API int nckv_delta_step(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *x, int64_t x_stride, const float *x0, const float *rate, const void *b, int64_t b_stride,
+                      const void *gate, int64_t gate_stride, const float *norm_w, float eps, void *out, float *state, int B,
+                      int H, int G, int Dk, int Dv, int f32, void *stream);
+NCKV_API size_t nckv_route_workspace_bytes(int rows, int E, int top);
+NCKV_API int nckv_route(const float *logits, int32_t *offsets, int32_t *slot, float *scale, int rows, int E, int top,
+                      void *workspace, size_t workspace_bytes, void *stream);
+NCKV_API int nckv_experts(const void *a, const void *w, void *out, const int32_t *offsets, const int32_t *slot, const float *scale,
+                      int up, int R, int E, int top, int N, int K, int f32, int32_t *status, void *stream);
 
 #ifdef __cplusplus
 }

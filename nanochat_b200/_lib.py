@@ -60,12 +60,13 @@ SIGNATURES = {
     "nckv_flash_attn_fwd": (c_int, [c_void_p] * 5 + [c_int] * 6 + [c_void_p, c_void_p]),
     "nckv_flash_attn_bwd_workspace_bytes": (c_size_t, [c_int, c_int, c_int]),
     "nckv_flash_attn_bwd": (c_int, [c_void_p] * 10 + [c_int] * 6 + [c_void_p]),
-    "nckv_prefill_attn_split_p": (c_int, [c_void_p] * 5 + [c_int] * 6 + [c_i64, c_i64, c_int, c_void_p, c_void_p]),
-    "nckv_decode_attn_split_p": (c_int, [c_void_p] * 5 + [c_int] * 5 + [c_i64, c_i64, c_int, c_int, c_void_p, c_size_t,
-                                                          c_void_p]),
+    "nckv_prefill_attn_split_p": (c_int, [c_void_p] * 5 + [c_int] * 6 + [c_i64, c_i64, c_int, c_int, c_void_p, c_i64,
+                                                                                   c_void_p, c_void_p]),
+    "nckv_decode_attn_split_p": (c_int, [c_void_p] * 5 + [c_int] * 5 + [c_i64, c_i64, c_int, c_int, c_int, c_void_p, c_i64,
+                                                          c_void_p, c_size_t, c_void_p]),
     "nckv_rope_unit_append": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p] * 5 + [c_i64] * 4 + [c_int] * 11 +
                               [c_float, c_float, c_int, c_void_p, c_void_p]),
-    "nckv_window_attn": (c_int, [c_void_p] * 5 + [c_i64] * 4 + [c_int] * 8 + [c_float, c_int, c_void_p]),
+    "nckv_window_attn": (c_int, [c_void_p] * 5 + [c_i64] * 4 + [c_int] * 8 + [c_float, c_int, c_void_p, c_i64, c_int, c_void_p]),
     "nckv_recurrent_workspace_bytes": (c_size_t, [c_int] * 5),
     "nckv_recurrent": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64] + [c_void_p] * 4 +
                        [c_i64, c_void_p, c_float, c_void_p, c_i64, c_void_p] + [c_int] * 7 + [c_void_p, c_size_t, c_void_p]),
@@ -75,6 +76,19 @@ SIGNATURES = {
     "nckv_silu_mul": (c_int, [c_void_p, c_void_p, c_i64, c_int, c_int, c_void_p]),
     "nckv_tanh_split": (c_int, [c_void_p, c_void_p, c_i64, c_int, c_int, c_void_p]),
     "nckv_softcap": (c_int, [c_void_p, c_i64, c_float, c_void_p]),
+    "nckv_rms_rope_append": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p] * 7 + [c_i64] * 4 + [c_int] * 11 +
+                             [c_float, c_float, c_int, c_void_p, c_void_p]),
+    "nckv_hyper_norm": (c_int, [c_void_p] * 3 + [c_int, c_void_p, c_int] + [c_void_p] * 6 + [c_int] * 3 + [c_float, c_int, c_void_p]),
+    "nckv_short_conv": (c_int, [c_void_p, c_i64] + [c_void_p] * 5 + [c_int] * 6 + [c_void_p]),
+    "nckv_gated_scan": (c_int, [c_void_p, c_i64, c_void_p, c_i64] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p]),
+    "nckv_delta_workspace_bytes": (c_size_t, [c_int] * 4),
+    "nckv_delta_rule": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_i64, c_void_p, c_void_p] +
+                        [c_int] * 7 + [c_void_p, c_size_t, c_void_p]),
+    "nckv_delta_step": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_i64, c_void_p, c_i64,
+                                                            c_void_p, c_float, c_void_p, c_void_p] + [c_int] * 6 + [c_void_p]),
+    "nckv_route_workspace_bytes": (c_size_t, [c_int] * 3),
+    "nckv_route": (c_int, [c_void_p] * 4 + [c_int] * 3 + [c_void_p, c_size_t, c_void_p]),
+    "nckv_experts": (c_int, [c_void_p] * 6 + [c_int] * 7 + [c_void_p, c_void_p]),
 }
 
 ERROR_NAMES = {-1: "NCKV_E_ARG", -2: "NCKV_E_UNSUPPORTED", -3: "NCKV_E_CAPACITY", -4: "NCKV_E_CUDA"}

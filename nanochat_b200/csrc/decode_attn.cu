@@ -102,6 +102,7 @@ struct DecodeParams {
     int rec_floats;
     int W;                 // warps of the streaming grid (the run geometry depends on it)
     float scale_log2;
+    HeadEnd end;           // SPLIT_P form only
 };
 
 struct TileCursor {
@@ -683,8 +684,11 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmap_k,
             const bool complete = (seg_j0 == 0) && (cons.j == cons.nt - 1);
             const long long row_base = (long long)cons.b * p.Hq + (long long)cons.h * G;
             if (complete) {
-                const float inv0 = 1.f / l0;
-                const float inv1 = GHI ? 1.f / l1 : 0.f;
+                float inv0 = 1.f / l0, inv1 = GHI ? 1.f / l1 : 0.f;
+                if constexpr (SPLIT_P) {
+                    if (g < G) inv0 = p.end.factor(m_run[0], l0, cons.b, cons.h * G + g);
+                    if (GHI && g + 8 < G) inv1 = p.end.factor(m_run[1], l1, cons.b, cons.h * G + g + 8);
+                }
 #pragma unroll
                 for (int nd = 0; nd < 16; ++nd) {
                     const int d = nd * 8 + 2 * t4;
@@ -971,7 +975,7 @@ __global__ void __launch_bounds__(MERGE_WARPS * 32) decode_merge_kernel(const De
                          __ldcg(p.lse + item));
             continue;
         }
-        const float inv = 1.f / L;
+        const float inv = p.end.active() ? p.end.factor(M, L, item / p.Hq, item % p.Hq) : 1.f / L;
         acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
         const long long o = (long long)item * NCKV_D + lane * 4;
         uint2 packed;
@@ -1092,7 +1096,7 @@ static int decode_launch(const void *q, const void *k_cache, const void *v_cache
                          int64_t cache_batch_stride, int64_t cache_token_stride, int seqlen_offset, int window_left,
                          int kv_begin, int kv_end, nckv::KvSplit split, const nckv::PushDesc &push, void *workspace,
                          size_t workspace_bytes, void *stream, nckv::PagedDesc paged = nckv::PagedDesc{nullptr, 0, 0, 0},
-                         bool split_p = false) {
+                         bool split_p = false, nckv::HeadEnd end = nckv::HeadEnd{0, nullptr, 0}) {
     using namespace nckv;
     int rc0 = decode_check(q, k_cache, v_cache, cache_seqlens, out, out_f32, workspace, B, Hq, Hkv, D, T_max,
                            workspace_bytes);
@@ -1150,6 +1154,7 @@ static int decode_launch(const void *q, const void *k_cache, const void *v_cache
     p.rec_floats = rec_floats_for(G);
     p.W = grid * DEC_WARPS;
     p.scale_log2 = (float)(1.4426950408889634 / sqrt((double)D));
+    p.end = end;
 
     const size_t smem = decode_smem_bytes(B), smem_max = decode_smem_bytes(DEC_MAX_B);
     static bool attr_set[64] = {false};  // per device; setting the attribute twice from racing threads is harmless
@@ -1218,8 +1223,8 @@ int nckv_decode_attn(const void *q, const void *k_cache, const void *v_cache,
 
 int nckv_decode_attn_split_p(const void *q, const void *k_cache, const void *v_cache, const int32_t *cache_seqlens, void *out,
                              int B, int Hq, int Hkv, int D, int T_max, int64_t cache_batch_stride,
-                             int64_t cache_token_stride, int seqlen_offset, int window_left, void *workspace,
-                             size_t workspace_bytes, void *stream) {
+                             int64_t cache_token_stride, int seqlen_offset, int window_left, int sink, const void *gate,
+                             int64_t gate_stride, void *workspace, size_t workspace_bytes, void *stream) {
     if (!out) {
         nckv::set_error("decode_attn_split_p: null pointer argument");
         return NCKV_E_ARG;
@@ -1227,7 +1232,8 @@ int nckv_decode_attn_split_p(const void *q, const void *k_cache, const void *v_c
     nckv::PushDesc none = {};
     return decode_launch(q, k_cache, v_cache, cache_seqlens, out, nullptr, nullptr, B, Hq, Hkv, D, T_max,
                          cache_batch_stride, cache_token_stride, seqlen_offset, window_left, 0, 0,
-                         nckv::KvSplit{0, 0, 0}, none, workspace, workspace_bytes, stream, nckv::PagedDesc{nullptr, 0, 0, 0}, true);
+                         nckv::KvSplit{0, 0, 0}, none, workspace, workspace_bytes, stream, nckv::PagedDesc{nullptr, 0, 0, 0}, true,
+                         nckv::HeadEnd{sink, static_cast<const __nv_bfloat16 *>(gate), gate_stride});
 }
 
 int nckv_decode_attn_paged(const void *q, const void *k_pool, const void *v_pool, const int32_t *block_table,

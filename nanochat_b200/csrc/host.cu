@@ -112,6 +112,27 @@ int make_kv_tensor_map_5d(CUtensorMap *map, const void *base, int B, int T, int 
     return NCKV_OK;
 }
 
+int make_tensor_map(CUtensorMap *map, const void *base, int rank, const int64_t *dims, const int64_t *strides, const int *box) {
+    EncodeTiledFn fn = encode_tiled_fn();
+    if (!fn) return NCKV_E_CUDA;
+    cuuint64_t d[5], st[4];
+    cuuint32_t bx[5], estr[5];
+    for (int i = 0; i < rank; ++i) {
+        d[i] = (cuuint64_t)dims[i];
+        bx[i] = (cuuint32_t)box[i];
+        estr[i] = 1u;
+        if (i) st[i - 1] = (cuuint64_t)strides[i - 1] * 2;
+    }
+    CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (cuuint32_t)rank, const_cast<void *>(base), d, st, bx, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) {
+        set_error("cuTensorMapEncodeTiled failed with CUresult %d (rank %d)", (int)r, rank);
+        return NCKV_E_CUDA;
+    }
+    return NCKV_OK;
+}
+
 }  // namespace nckv
 
 extern "C" {

@@ -34,6 +34,10 @@ int make_kv_tensor_map(CUtensorMap *map, const void *base, int B, int T, int Hkv
 int make_kv_tensor_map_5d(CUtensorMap *map, const void *base, int B, int T, int Hkv,
                           int64_t batch_stride, int64_t token_stride, int box_tokens);
 
+// A bf16 tensor of `rank` dimensions (innermost first, strides in elements for dimensions 1 ..) as a tiled tensor
+// map with the 128-byte swizzle; elements outside read as zero.
+int make_tensor_map(CUtensorMap *map, const void *base, int rank, const int64_t *dims, const int64_t *strides, const int *box);
+
 // ---- sequence-split bookkeeping (shared by host checks and kernels) ---------------------------
 // Block-cyclic ownership of key positions: position p belongs to shard (p / block) % world and
 // sits at local index (p / (block*world)) * block + p % block there.  owned_below(n) = how many
@@ -56,6 +60,23 @@ struct PeerPtrs {
     float *buf[NCKV_MAX_PEERS];
 };
 __host__ __device__ inline long long p2p_per_floats(int rows) { return (long long)rows * NCKV_D + ((rows + 3) & ~3); }
+
+// What a head's softmax ends with besides the division by its sum: a sink (one more term of score 0 in the
+// sum, without a value) and a sigmoid gate per token and head.
+struct HeadEnd {
+    int sink;
+    const __nv_bfloat16 *gate;  // rows of one logit per head, or null
+    long long gate_stride;
+    __host__ __device__ bool active() const { return sink || gate; }
+#ifdef __CUDACC__
+    // factor on the unnormalised output; max and sum of the exponentials in powers of two
+    __device__ __forceinline__ float factor(float m, float l, long long row, int head) const {
+        float f = 1.f / (sink ? l + exp2f(-m) : l);
+        if (gate) f *= 1.f / (1.f + __expf(-__bfloat162float(gate[row * gate_stride + head])));
+        return f;
+    }
+#endif
+};
 
 // ---- device helpers ----------------------------------------------------------------------
 #ifdef __CUDACC__
@@ -159,6 +180,22 @@ __device__ __forceinline__ void tma_load_4d(void *smem_dst, const CUtensorMap *m
         "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes"
         " [%0], [%1, {%2, %3, %4, %5}], [%6];" ::"r"(smem_u32(smem_dst)),
         "l"(map), "r"(c0), "r"(c1), "r"(c2), "r"(c3), "r"(smem_u32(bar))
+        : "memory");
+}
+__device__ __forceinline__ void tma_load_2d(void *smem_dst, const CUtensorMap *map, uint64_t *bar, int c0, int c1) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes"
+        " [%0], [%1, {%2, %3}], [%4];" ::"r"(smem_u32(smem_dst)),
+        "l"(map), "r"(c0), "r"(c1), "r"(smem_u32(bar))
+        : "memory");
+}
+// Four rows of a 2-D map whose box is one row high, one after the other in shared memory.
+__device__ __forceinline__ void tma_gather4(void *smem_dst, const CUtensorMap *map, uint64_t *bar, int c0, int r0, int r1,
+                                            int r2, int r3) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes"
+        " [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(smem_u32(smem_dst)),
+        "l"(map), "r"(c0), "r"(r0), "r"(r1), "r"(r2), "r"(r3), "r"(smem_u32(bar))
         : "memory");
 }
 // Same, with an L2 cache policy (e.g. evict-first for data that is streamed once).

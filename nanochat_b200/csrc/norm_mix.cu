@@ -14,7 +14,7 @@
 //   silu_mul_kernel     out = T(silu(gate) * up) over rows [gate | up]
 //   tanh_split_kernel   tanh of a fp32 row as bf16 hi | lo halves (their sum carries 16 bits), or as fp32
 //   softcap_kernel      cap * tanh(z / cap), fp32 in place
-#include "nckv_common.cuh"
+#include "vec_io.cuh"
 
 namespace nckv {
 
@@ -36,48 +36,6 @@ struct ResidNormParams {
     int B, T, W, run, n_mix, vocab;
     float eps;
 };
-
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ void put(float *p, float v) { *p = v; }
-__device__ __forceinline__ void put(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
-
-// V consecutive elements
-__device__ __forceinline__ void get_v(const float *p, float (&o)[1]) { o[0] = p[0]; }
-__device__ __forceinline__ void get_v(const __nv_bfloat16 *p, float (&o)[1]) { o[0] = to_f(p[0]); }
-__device__ __forceinline__ void get_v(const float *p, float (&o)[4]) {
-    const float4 f = *reinterpret_cast<const float4 *>(p);
-    o[0] = f.x; o[1] = f.y; o[2] = f.z; o[3] = f.w;
-}
-__device__ __forceinline__ void get_v(const __nv_bfloat16 *p, float (&o)[4]) {
-    const uint2 f = *reinterpret_cast<const uint2 *>(p);
-    o[0] = bf16lo(f.x); o[1] = bf16hi(f.x); o[2] = bf16lo(f.y); o[3] = bf16hi(f.y);
-}
-__device__ __forceinline__ void put_v(float *p, const float (&o)[1]) { p[0] = o[0]; }
-__device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[1]) { put(p, o[0]); }
-__device__ __forceinline__ void put_v(float *p, const float (&o)[4]) {
-    *reinterpret_cast<float4 *>(p) = make_float4(o[0], o[1], o[2], o[3]);
-}
-__device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[4]) {
-    *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]));
-}
-
-__device__ __forceinline__ void get_v(const float *p, float (&o)[8]) {
-    const float4 a = reinterpret_cast<const float4 *>(p)[0], b = reinterpret_cast<const float4 *>(p)[1];
-    o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
-}
-__device__ __forceinline__ void get_v(const __nv_bfloat16 *p, float (&o)[8]) {
-    const uint4 f = *reinterpret_cast<const uint4 *>(p);
-    o[0] = bf16lo(f.x); o[1] = bf16hi(f.x); o[2] = bf16lo(f.y); o[3] = bf16hi(f.y);
-    o[4] = bf16lo(f.z); o[5] = bf16hi(f.z); o[6] = bf16lo(f.w); o[7] = bf16hi(f.w);
-}
-__device__ __forceinline__ void put_v(float *p, const float (&o)[8]) {
-    reinterpret_cast<float4 *>(p)[0] = make_float4(o[0], o[1], o[2], o[3]);
-    reinterpret_cast<float4 *>(p)[1] = make_float4(o[4], o[5], o[6], o[7]);
-}
-__device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[8]) {
-    *reinterpret_cast<uint4 *>(p) = make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
-}
 
 __device__ __forceinline__ float block_sum(float v, float *s_part) {
 #pragma unroll

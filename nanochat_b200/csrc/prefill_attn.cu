@@ -67,6 +67,7 @@ struct PrefillParams {
     int n_groups;     // the last group takes the remaining pairs (fewer than 2 group_pairs)
     int window_left;
     float scale_log2;
+    HeadEnd end;      // SPLIT_P form only
 };
 
 // One work item: PF_M query tokens of one (row, q head) and the key tiles they see.
@@ -490,7 +491,9 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
                 }
                 tc_fence_after();
             }
-            const float inv = (n_tiles > 0 && l_run > 0.f) ? 1.f / l_run : 0.f;
+            float inv = (n_tiles > 0 && l_run > 0.f) ? 1.f / l_run : 0.f;
+            if constexpr (SPLIT_P)
+                if (inv > 0.f && tq < p.T_new) inv = p.end.factor(m_used, l_run, (long long)it.b * p.T_new + tq, it.hq);
             if (p.lse && tq < p.T_new)  // m_used and l_run are in powers of two
                 p.lse[((long long)it.b * p.Hq + it.hq) * p.T_new + tq] =
                     (n_tiles > 0 && l_run > 0.f) ? (m_used + log2f(l_run)) * 0.6931471805599453f : -INFINITY;
@@ -538,7 +541,7 @@ static size_t prefill_smem_bytes() {
 static int prefill_launch(const void *q, const void *k, const void *v, const int32_t *cache_seqlens, void *out,
                           float *lse, int B, int T_new, int Hq, int Hkv, int D, int T_k, int64_t kv_batch_stride,
                           int64_t kv_token_stride, int window_left, int32_t *status, void *stream,
-                          bool split_p = false) {
+                          bool split_p = false, nckv::HeadEnd end = nckv::HeadEnd{0, nullptr, 0}) {
     using namespace nckv;
     const auto kernel = split_p ? prefill_attn_kernel<true> : prefill_attn_kernel<false>;
     if (!q || !k || !v || !out || !status) {
@@ -586,6 +589,7 @@ static int prefill_launch(const void *q, const void *k, const void *v, const int
     p.B = B; p.T_new = T_new; p.Hq = Hq; p.Hkv = Hkv; p.T_k = T_k;
     p.window_left = window_left;
     p.scale_log2 = (float)(1.4426950408889634 / sqrt((double)D));
+    p.end = end;
     const int n_items = n_qtiles * Hq * B;
     const int grid = n_items < 2 * sm_count() ? n_items : 2 * sm_count();  // two CTAs per SM, persistent
     p.n_qtiles = n_qtiles;
@@ -650,9 +654,10 @@ extern "C" int nckv_prefill_attn(const void *q, const void *k, const void *v, co
 extern "C" int nckv_prefill_attn_split_p(const void *q, const void *k, const void *v, const int32_t *cache_seqlens,
                                          void *out, int B, int T_new, int Hq, int Hkv, int D, int T_k,
                                          int64_t kv_batch_stride, int64_t kv_token_stride, int window_left,
-                                         int32_t *status, void *stream) {
+                                         int sink, const void *gate, int64_t gate_stride, int32_t *status, void *stream) {
     return prefill_launch(q, k, v, cache_seqlens, out, nullptr, B, T_new, Hq, Hkv, D, T_k, kv_batch_stride,
-                          kv_token_stride, window_left, status, stream, true);
+                          kv_token_stride, window_left, status, stream, true,
+                          nckv::HeadEnd{sink, static_cast<const __nv_bfloat16 *>(gate), gate_stride});
 }
 
 // Forward of flash_attn_func for training: the same kernel over plain (B, T, H, D) tensors, which also

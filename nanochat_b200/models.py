@@ -13,7 +13,7 @@ import torch
 from .weights import read_safetensors
 
 _REGISTRY = {}
-_MODULES = ("gpt", "sipadra")  # imported on first use; each registers its classes
+_MODULES = ("gpt", "sipadra", "zuvulorn")  # imported on first use; each registers its classes
 
 
 def register(name):

@@ -5,14 +5,13 @@ mixing, ``parallel``: windowed attention beside scaled linear attention) and the
 feed-forward, if it has one.  Sublayers read the stream itself.  The output head is the embedding
 table, with a soft cap on the logits.  Sizes come from the configuration or the tensors' shapes.
 """
-import contextlib
 from dataclasses import dataclass, field
 from typing import List, Optional
 
 import torch
 
 from . import mixer_ops as mo
-from .engine import HybridCache
+from .hybrid import HybridDecoder, Scope
 from .mixers import GatedFeedForward, ParallelMixer, Rotary, ScaledLinearAttention, WindowAttention, WkvMixer, f32
 from .models import register
 
@@ -68,56 +67,29 @@ def tensor_shapes(config, rank):
     return shapes
 
 
-class _Scope:
-    """The tensors below a name prefix, looked up without it."""
-
-    def __init__(self, tensors, prefix):
-        self.tensors, self.prefix = tensors, prefix
-
-    def __getitem__(self, name):
-        return self.tensors[self.prefix + name]
-
-
 class _Layer:
     def __init__(self, i, spec, tensors, eps, dtype):
         p, m = f"l{i}.", spec["mixer"]
-        mix = _Scope(tensors, p + "mix.")
+        mix = Scope(tensors, p + "mix.")
         if spec["type"] == "wkv":
             self.mixer = WkvMixer(p + "wkv", m["heads"], m["dim"], mix, eps, dtype)
         else:
             a, b = m["left"], m["right"]
             left = WindowAttention(p + "left", a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"], a["scale"],
                                    Rotary(a["rot"]["dims"], a["rot"]["base"], a["rot"].get("scaling")),
-                                   _Scope(tensors, p + "mix.left."), eps, dtype)
+                                   Scope(tensors, p + "mix.left."), eps, dtype)
             right = ScaledLinearAttention(p + "right", b["heads"], b["dim"], b["vdim"], b["decay"],
-                                          _Scope(tensors, p + "mix.right."), eps, dtype)
+                                          Scope(tensors, p + "mix.right."), eps, dtype)
             self.mixer = ParallelMixer(left, right, m["left_scale"], m["right_scale"])
         self.norm1 = f32(tensors[p + "norm1"])
         self.ff = self.norm2 = None
         if spec.get("mlp") is not None:
-            self.ff = GatedFeedForward(_Scope(tensors, p + "mlp."))
+            self.ff = GatedFeedForward(Scope(tensors, p + "mlp."))
             self.norm2 = f32(tensors[p + "norm2"])
 
 
-@contextlib.contextmanager
-def _full_precision_sums():
-    """bf16 products keep fp32 partial sums, fp32 products stay fp32 (no TF32)."""
-    m = torch.backends.cuda.matmul
-    saved = m.allow_bf16_reduced_precision_reduction, m.allow_tf32
-    m.allow_bf16_reduced_precision_reduction, m.allow_tf32 = False, False
-    try:
-        yield
-    finally:
-        m.allow_bf16_reduced_precision_reduction, m.allow_tf32 = saved
-
-
 @register("Sipadra")
-class Sipadra:
-    """Inference model with GPT's interface: ``config``, ``get_device``, ``make_cache``,
-    ``forward(ids, kv_cache=...)``."""
-
-    accepts_logits_at = True
-
+class Sipadra(HybridDecoder):
     def __init__(self, config, tensors, dtype=torch.bfloat16):
         self.config, self.dtype = config, dtype
         self.embed = tensors["embed"]
@@ -126,40 +98,16 @@ class Sipadra:
         self.layers = [_Layer(i, spec, tensors, config.eps, dtype) for i, spec in enumerate(config.layers)]
         self.final_norm = f32(tensors["final.norm"])
 
-    @classmethod
-    def from_dict(cls, config, tensors, dtype, device):
-        parsed = SipadraConfig.from_dict(config)
-        for name, shape in tensor_shapes(config, rank=None).items():
-            if name not in tensors:
-                raise ValueError(f"the weights lack {name}")
-            have = tuple(tensors[name].shape)
-            if len(have) != len(shape) or any(want not in (None, n) for want, n in zip(shape, have)):
-                raise ValueError(f"{name} is {have}, the configuration says {shape}")
-        tensors = {k: v.to(device=device, dtype=dtype) for k, v in tensors.items()}
-        return cls(parsed, tensors, dtype)
-
-    def get_device(self):
-        return self.embed.device
-
-    def make_cache(self, batch_size, seq_len, page_tokens=None, n_pages=None):
-        if page_tokens:
-            raise NotImplementedError("this model keeps its keys and states in dense rows; page_tokens is not supported")
-        cache = HybridCache(batch_size, seq_len, self.get_device())
-        for layer in self.layers:
-            layer.mixer.declare(cache)
-        return cache
+    parse = staticmethod(SipadraConfig.from_dict)
+    shapes = staticmethod(lambda config: tensor_shapes(config, rank=None))
 
     @torch.inference_mode()
     def forward(self, idx, targets=None, kv_cache=None, logits_at=None, on_layer=None):
         """fp32 logits (B, T, vocab), or (B, len(logits_at), vocab) at the given places of the T tokens (an
         empty list runs the tokens and returns None).  ``on_layer(i, x)`` sees the stream after each layer."""
-        if targets is not None:
-            raise NotImplementedError("this model is inference-only")
-        B, T = idx.shape
+        B, T, kv_cache = self.begin(idx, targets, kv_cache)
         cfg = self.config
-        if kv_cache is None:
-            kv_cache = self.make_cache(B, T)
-        with _full_precision_sums():
+        with mo.full_precision_sums():
             x = y = w = None
             common = dict(eps=cfg.eps, dtype=self.dtype, B=B, T=T)
             source = dict(tokens=idx.contiguous().view(-1), table=self.embed)
@@ -184,9 +132,7 @@ class Sipadra:
                 if len(logits_at) == 0:
                     return None
                 n = len(logits_at)
-                rows = torch.as_tensor(logits_at, device=x.device)
-                x = x.view(B, T, -1).index_select(1, rows).contiguous()
-                y = y.view(B, T, -1).index_select(1, rows).contiguous()
+                x, y = self.pick(x, B, T, logits_at), self.pick(y, B, T, logits_at)
             _, h, _ = mo.resid_norm(x, y, w, eps=cfg.eps, dtype=self.dtype, B=B, T=n, final_weight=self.final_norm)
             logits = mo.product(h, self.embed, f32_out=True)
             if cfg.logit_softcap is not None:
