@@ -1062,12 +1062,12 @@ def _time_cold(fn, iters, flush, warmup=3):
     return sorted(times)[len(times) // 2]
 
 
-def sipadra_models(dev, iters):
-    """Whole-model prefill and decode tokens/s of both designs."""
+def design_models(dev, iters, builders):
+    """Whole-model prefill and decode tokens/s of some designs, (name, function (size, device) -> model)."""
     from nanochat_b200.engine import GraphedDecodeStep, new_cache
     rows = []
     for name in SIPADRA_SIZES:
-        for kind, build in (("sipadra", build_sipadra), ("gpt", build_gpt_like)):
+        for kind, build in builders:
             model = build(name, dev)
             for Bc, T in ((1, 2048), (1, 8192), (8, 2048)):
                 cache = new_cache(model, Bc, T, torch.bfloat16)
@@ -1101,6 +1101,20 @@ def sipadra_models(dev, iters):
     return rows
 
 
+class KernelTable:
+    """Times of single kernels against their rooflines."""
+
+    def __init__(self, dev, iters, peak):
+        self.rows, self.iters, self.peak = [], iters, peak
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def __call__(self, kernel, shape, fn, nbytes=0, flops=0, peak_flops=None):
+        sec = _time_cold(fn, self.iters, self.flush)
+        need = max(nbytes / (self.peak * 1e9), flops / (peak_flops * 1e12) if flops else 0)
+        self.rows.append({"kernel": kernel, "shape": shape, "us": sec * 1e6, "roofline_us": need * 1e6, "frac": need / sec,
+                          "bound": "bytes" if nbytes / (self.peak * 1e9) >= need else "flops"})
+
+
 def sipadra_kernels(dev, iters, peak, tflops):
     """Kernels of the design, and the GPT path's like kernels on the same sizes, against their rooflines."""
     from nanochat_b200 import mixer_ops as mo, ops
@@ -1109,14 +1123,7 @@ def sipadra_kernels(dev, iters, peak, tflops):
     bf, f32 = torch.bfloat16, torch.float32
     gen = torch.Generator(device=dev).manual_seed(12)
     rnd = lambda *shape, dtype=bf: torch.randn(*shape, generator=gen, device=dev).to(dtype)
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    rows = []
-
-    def note(kernel, shape, fn, nbytes=0, flops=0, peak_flops=None):
-        sec = _time_cold(fn, iters, flush)
-        need = max(nbytes / (peak * 1e9), flops / (peak_flops * 1e12) if flops else 0)
-        rows.append({"kernel": kernel, "shape": shape, "us": sec * 1e6, "roofline_us": need * 1e6, "frac": need / sec,
-                     "bound": "bytes" if nbytes / (peak * 1e9) >= need else "flops"})
+    note = KernelTable(dev, iters, peak)
 
     for name, size in SIPADRA_SIZES.items():
         W, H, D = size["width"], size["wkv_heads"], 64
@@ -1174,10 +1181,141 @@ def sipadra_kernels(dev, iters, peak, tflops):
             else:
                 note("gpt: prefill_attention", shape, lambda: ops.prefill_attention(q4, kc, vc, lens, win - 1), nb, fl, tflops)
             del r, k, v, g, x, st, z, o32, xs, y, gu, h4, kc, vc, qkv, q4, k4, v4
-    return rows
+    return note.rows
 
 
-def run_sipadra_case(args):
+# ------------------------------------------------------------------------------------------------
+# Zuvulorn (rglru, channel_delta and attention layers with experts) beside the Sipadra of equal width and depth
+# ------------------------------------------------------------------------------------------------
+ZUVULORN_SIZES = {
+    # `top` experts of `ff` are as many weights per token as Sipadra's feed-forward of the same size has
+    "d24": dict(width=1536, n_layer=24, ff=1024, experts=16, top=4, blocks=12, delta=(12, 12), attn=(12, 12), rank=64),
+    "d32": dict(width=2048, n_layer=32, ff=1376, experts=16, top=4, blocks=16, delta=(16, 16), attn=(16, 4), rank=96),
+}
+ZUVULORN_STREAMS, ZUVULORN_TAPS = 4, 4
+
+
+def zuvulorn_config(width, n_layer, ff, experts, top, blocks, delta, attn, rank, vocab=32768):
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    layers = []
+    for i in range(n_layer):
+        if i % 3 == 0:
+            mixer = "rglru", {"width": width, "blocks": blocks, "conv": ZUVULORN_TAPS}
+        elif i % 3 == 1:
+            mixer = "channel_delta", {"heads": delta[0], "kv_heads": delta[1], "dim": 128, "vdim": 128, "conv": ZUVULORN_TAPS}
+        else:
+            mixer = "attention", {"heads": attn[0], "kv_heads": attn[1], "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                  "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+            if i % 6 == 5:
+                mixer[1]["kv_from"] = i - 3
+        layers.append({"type": mixer[0], "mixer": mixer[1], "mlp": mlp})
+    return {"architecture": "Zuvulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": ZUVULORN_STREAMS, "layers": layers}
+
+
+def build_zuvulorn(name, dev):
+    from nanochat_b200.zuvulorn import Zuvulorn, tensor_shapes
+    size = ZUVULORN_SIZES[name]
+    cfg = zuvulorn_config(**size)
+    gen = torch.Generator(device=dev).manual_seed(11)
+    tensors = {}
+    for key, shape in tensor_shapes(cfg, size["rank"]).items():
+        z = torch.randn(shape, generator=gen, device=dev)
+        if "norm" in key:
+            z = 1 + 0.1 * z
+        elif ".hc" in key:
+            z = torch.eye(shape[0], device=dev) if key.endswith(".mix") else torch.ones(shape, device=dev) / shape[0]
+        elif key.endswith(("lam", "A_log", "dt_bias")):
+            z = z - 2
+        elif key != "embed":
+            z = z * shape[-1] ** -0.5
+        tensors[key] = z.to(torch.bfloat16)
+    return Zuvulorn.from_dict(cfg, tensors, torch.bfloat16, dev)
+
+
+def zuvulorn_kernels(dev, iters, peak, tflops):
+    """Kernels of the design, and Sipadra's (or the dense feed-forward's) like kernels on the same sizes, against their rooflines."""
+    from nanochat_b200 import mixer_ops as mo
+    from nanochat_b200.mixers import rotary_table
+    bf, f32 = torch.bfloat16, torch.float32
+    gen = torch.Generator(device=dev).manual_seed(12)
+    rnd = lambda *shape, dtype=bf: torch.randn(*shape, generator=gen, device=dev).to(dtype)
+    note = KernelTable(dev, iters, peak)
+    for name, size in ZUVULORN_SIZES.items():
+        W, S, K, D = size["width"], ZUVULORN_STREAMS, ZUVULORN_TAPS, 128
+        H, G = size["delta"]
+        Hq, Hkv = size["attn"]
+        E, top, ff, blocks = size["experts"], size["top"], size["ff"], size["blocks"]
+        norm_d, vec = rnd(D, dtype=f32), lambda n: rnd(n, dtype=f32)
+        w_in, w_down = rnd(E, 2 * ff, W), rnd(E, W, ff)
+        dense_in, dense_down = rnd(2 * top * ff, W), rnd(W, top * ff)
+        for Bc, T in ((1, 2048), (1, 8192), (8, 2048), (64, 1), (256, 1)):
+            N, shape = Bc * T, f"{name} B{Bc} T{T}"
+            # streams
+            xs, y, y_top, w = rnd(N, S, W, dtype=f32), rnd(N, W), rnd(N, top, W), vec(W)
+            back, into = (torch.eye(S, device=dev), torch.ones(S, device=dev)), torch.ones(S, device=dev)
+            note("hyper_norm", shape, lambda: mo.hyper_norm(xs, y, back, into, w, 1e-6, bf), N * W * (8 * S + 4))
+            note("hyper_norm + experts' sum", shape, lambda: mo.hyper_norm(xs, y_top, back, into, w, 1e-6, bf), N * W * (8 * S + 2 + 2 * top))
+            x1 = rnd(N, W, dtype=f32)
+            note("sipadra: resid_norm", shape, lambda: mo.resid_norm(x1, y, w, 1e-6, bf, Bc, T, want_h=True), N * W * 12)
+            del xs, y_top, x1
+            # convolution and real-gated recurrence
+            z = rnd(N, 2 * W)
+            zy, zx = z.split([W, W], 1)
+            taps, carry = rnd(K, W, dtype=f32), torch.zeros(Bc, K - 1, W, device=dev)
+            note("short_conv", shape, lambda: mo.short_conv(zx, taps, carry, Bc, T, taps[0], taps[0]), N * W * 4 + 8 * carry.numel())
+            gates, rate, st = rnd(blocks, N, 2 * W // blocks, dtype=f32), vec(W).abs() * 0.1, torch.zeros(Bc, W, device=dev)
+            gb = rnd(2, W, dtype=f32)
+            note("gated_scan", shape, lambda: mo.gated_scan(zx, zy, gates, gb, gb[0], rate, st, Bc, T), N * W * 14 + 8 * st.numel())
+            del z, zy, zx, gates
+            # delta rule, and the recurrence without corrections of equal heads
+            q, k, v, g = (rnd(N, H * D) for _ in range(4))
+            x, beta = rnd(N, H * D, dtype=f32), rnd(N, H)
+            st = torch.zeros(Bc, H, D, D, device=dev)
+            dt, dr = vec(H * D) - 2, vec(H).exp()
+            note("delta_rule", shape, lambda: mo.delta_rule(q, k, v, x, dt, dr, beta, st, Bc, T, H, H, D, D, g, norm_d, 1e-6),
+                 N * H * D * 14 + 8 * st.numel(), 8 * N * H * D * D, FP32_TFLOPS)
+            nw = norm_d.repeat(H)
+            note("sipadra: recurrent wkv", shape, lambda: mo.recurrent(q, k, v, st, Bc, T, H, D, D, decay_logits=x, decay_bias=dt, bonus=dt,
+                 gate=g, norm_weight=nw, eps=1e-6), N * H * D * 14 + 8 * st.numel(), 6 * N * H * D * D, FP32_TFLOPS)
+            del q, k, v, g, x, st
+            # attention
+            ctx = 1024 if T == 1 else 0
+            cap = ctx + T
+            kc, vc = rnd(Bc, cap, Hkv, D), rnd(Bc, cap, Hkv, D)
+            lens = torch.full((Bc,), cap - T, dtype=torch.int32, device=dev)
+            qkv = rnd(N, (Hq + 2 * Hkv) * D)
+            lq, lk, lv = qkv.split([Hq * D, Hkv * D, Hkv * D], 1)
+            table, wq, wk, hg = rotary_table(cap, D, 5e5, None, dev), vec(Hq * D), vec(Hkv * D), rnd(N, Hq)
+            ab = N * (Hq + 2 * Hkv) * 4 * D + cap * 4 * D
+            note("rms_rope_append", shape, lambda: mo.rms_rope_append(lq, lk, lv, wq, wk, table, D, kc, vc, lens, Bc, T, Hq, Hkv, D, D, 1.0, 1e-6), ab)
+            note("sipadra: rope_unit_append", shape, lambda: mo.rope_unit_append(lq, lk, lv, table, D, kc, vc, lens, Bc, T, Hq, Hkv, D, D, 1.0, 1e-6), ab)
+            q4 = lq.contiguous().view(Bc, T, Hq, D)
+            if T == 1:
+                nb, fl = 4 * Bc * Hkv * D * cap + 4 * N * Hq * D, 0
+            else:
+                nb, fl = 4 * N * (Hq + Hkv) * D, 4 * D * Bc * Hq * (T * (T + 1) // 2)
+            note("attention + sink + gate", shape, lambda: mo.split_p_attention(q4, kc, vc, lens, None, sink=True, gate=hg), nb, fl, tflops)
+            note("sipadra: split_p attention", shape, lambda: mo.split_p_attention(q4, kc, vc, lens, None), nb, fl, tflops)
+            del kc, vc, qkv, lq, lk, lv, q4
+            # experts, and the dense feed-forward with as many weights per token
+            h, logits = rnd(N, W), rnd(N, E, dtype=f32)
+            with mo.full_precision_sums():
+                note("routing", shape, lambda: mo.Routing(logits, top), N * (4 * E + 8 * top))
+                r = mo.Routing(logits, top)
+                used = int((r.offsets[1:] > r.offsets[:-1]).sum())
+                R = N * top
+                act = mo.expert_product(h, w_in, r, True)
+                note("experts up", shape, lambda: mo.expert_product(h, w_in, r, True), used * 4 * ff * W + 2 * N * W + 2 * R * ff, 4 * R * W * ff, tflops)
+                note("experts down", shape, lambda: mo.expert_product(act, w_down, r, False), used * 2 * ff * W + 2 * R * (W + ff), 2 * R * W * ff, tflops)
+                note("sipadra: dense up + silu_mul", shape, lambda: mo.silu_mul(mo.product(h, dense_in)),
+                     4 * top * ff * W + 2 * N * W + 10 * R * ff, 4 * R * W * ff, tflops)
+                gu = mo.silu_mul(mo.product(h, dense_in))
+                note("sipadra: dense down", shape, lambda: mo.product(gu, dense_down), 2 * top * ff * W + 2 * N * W + 2 * R * ff, 2 * R * W * ff, tflops)
+            del h, logits, r, act, gu
+    return note.rows
+
+
+def run_design_case(args):
     from nanochat_b200 import ops
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
@@ -1189,13 +1327,19 @@ def run_sipadra_case(args):
         tflops = 1590.0
     iters = min(max(args.steps, 5), 20)
     out = {"case": args.case, "n_gpus": 1, "data": "synthetic", "dtype": "bf16", "peak_gbs": peak, "peak_tflops": tflops,
-           "peak_kind": f"of {kind}", "fp32_tflops_nominal": FP32_TFLOPS, "sizes": SIPADRA_SIZES, "iters": iters}
+           "peak_kind": f"of {kind}", "fp32_tflops_nominal": FP32_TFLOPS, "iters": iters}
+    if args.case.startswith("sipadra"):
+        builders, kernels = (("sipadra", build_sipadra), ("gpt", build_gpt_like)), sipadra_kernels
+        out["sizes"] = SIPADRA_SIZES
+    else:
+        builders, kernels = (("zuvulorn", build_zuvulorn), ("sipadra", build_sipadra)), zuvulorn_kernels
+        out["sizes"] = ZUVULORN_SIZES
     sampler = ClockSampler(0)
     sampler.start()
     with torch.no_grad():
-        if args.case == "sipadra":
-            out["models"] = sipadra_models(dev, iters)
-        out["kernels"] = sipadra_kernels(dev, iters, peak, tflops)
+        if not args.case.endswith("_kernels"):
+            out["models"] = design_models(dev, iters, builders)
+        out["kernels"] = kernels(dev, iters, peak, tflops)
     out["clocks"] = sampler.stop()
     out["device_status"] = ops.read_status(dev)
     print(json.dumps(out), flush=True)
@@ -1215,12 +1359,13 @@ def main():
     ap.add_argument("--case", default=None,
                     help="secondary op-level measurement instead of the headline workload: decode_long, decode_gqa, "
                          "decode_gqa_window, decode_d24, decode_paged, prefill, prefill_paged, train_attn, broadcast, append, engine_d24, engine_d24_small, engine_d32, "
-                         "engine_d32_small, engine_api_d24, engine_api_small; sipadra (both models and kernels), sipadra_kernels")
+                         "engine_d32_small, engine_api_d24, engine_api_small; sipadra, zuvulorn (models and kernels beside the closest design's), "
+                         "sipadra_kernels, zuvulorn_kernels")
     args = ap.parse_args()
     global REGIONS_OVERRIDE
     REGIONS_OVERRIDE = args.regions
-    if args.case in ("sipadra", "sipadra_kernels"):
-        run_sipadra_case(args)
+    if args.case in ("sipadra", "sipadra_kernels", "zuvulorn", "zuvulorn_kernels"):
+        run_design_case(args)
     elif args.case:
         run_case(args)
     elif args.impl == "reference":

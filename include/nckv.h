@@ -430,7 +430,8 @@ NCKV_API int nckv_glue_ve_gate(const void *v, int64_t v_row_stride, const void *
  * nckv_delta_rule, nckv_delta_step: S <- diag(exp(-rate softplus(x + x0))) S; u = sigmoid(b) (v - S^T k);
  *   S <- S + k u^T; o = S^T q with q, k divided by sqrt(sum of squares + 1e-6) and q by sqrt(Dk).  H heads, G of
  *   them for q and k.  The rule leaves o as (B * T, H * Dv) fp32 (Dk <= 256); the step takes one token per row
- *   and leaves o / rms(o) * norm_w * sigmoid(gate) (Dv <= 128).
+ *   and leaves o / rms(o) * norm_w * sigmoid(gate) (Dv <= 128).  nckv_delta_chunk is the rule for bf16 on matrix
+ *   instructions with every fp32 operand in two tf32 terms (Dk <= 128).
  * nckv_route: per row the `top` largest of E logits; (row, choice) pairs sorted by expert: slot[i] = row * top +
  *   choice, scale[i] = sigmoid(logit), expert e at [offsets[e], offsets[e + 1]).
  * nckv_experts: up: out[i] = silu(s g) * (s u), [g; u] = w[e] a[slot[i] / top], s = scale[i], w (E, 2 N, K);
@@ -480,12 +481,18 @@ NCKV_API int nckv_short_conv(const void *x, int64_t x_stride, const float *taps,
                       void *out, int B, int T, int C, int K, int act, int f32, void *stream);
 NCKV_API int nckv_gated_scan(const void *u, int64_t u_stride, const void *y, int64_t y_stride, const float *gates,
                       const float *gate_bias, const float *y_bias, const float *rate, float *state, void *out, int B, int T,
-                      int C, int blocks, int f32, void *stream);
+                      int C, int blocks, int f32, void *workspace, size_t workspace_bytes, void *stream);
+NCKV_API size_t nckv_gated_scan_workspace_bytes(int B, int T, int C);
 NCKV_API size_t nckv_delta_workspace_bytes(int B, int T, int H, int Dk);
 NCKV_API int nckv_delta_rule(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                       const float *x, int64_t x_stride, const float *x0, const float *rate, const void *b, int64_t b_stride,
                       float *out, float *state, int B, int T, int H, int G, int Dk, int Dv, int f32, void *workspace,
                       size_t workspace_bytes, void *stream);
+NCKV_API size_t nckv_delta_chunk_workspace_bytes(int B, int T, int H, int Dk);
+NCKV_API int nckv_delta_chunk(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                      const float *x, int64_t x_stride, const float *x0, const float *rate, const void *b, int64_t b_stride,
+                      float *out, float *state, int B, int T, int H, int G, int Dk, int Dv, void *workspace,
+                      size_t workspace_bytes, int32_t *status, void *stream);
 NCKV_API int nckv_delta_step(const void *q, const void *k, const void *v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                       const float *x, int64_t x_stride, const float *x0, const float *rate, const void *b, int64_t b_stride,
                       const void *gate, int64_t gate_stride, const float *norm_w, float eps, void *out, float *state, int B,

@@ -80,10 +80,14 @@ SIGNATURES = {
                              [c_float, c_float, c_int, c_void_p, c_void_p]),
     "nckv_hyper_norm": (c_int, [c_void_p] * 3 + [c_int, c_void_p, c_int] + [c_void_p] * 6 + [c_int] * 3 + [c_float, c_int, c_void_p]),
     "nckv_short_conv": (c_int, [c_void_p, c_i64] + [c_void_p] * 5 + [c_int] * 6 + [c_void_p]),
-    "nckv_gated_scan": (c_int, [c_void_p, c_i64, c_void_p, c_i64] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p]),
+    "nckv_gated_scan": (c_int, [c_void_p, c_i64, c_void_p, c_i64] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p, c_size_t, c_void_p]),
+    "nckv_gated_scan_workspace_bytes": (c_size_t, [c_int] * 3),
     "nckv_delta_workspace_bytes": (c_size_t, [c_int] * 4),
     "nckv_delta_rule": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_i64, c_void_p, c_void_p] +
                         [c_int] * 7 + [c_void_p, c_size_t, c_void_p]),
+    "nckv_delta_chunk_workspace_bytes": (c_size_t, [c_int] * 4),
+    "nckv_delta_chunk": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_i64, c_void_p, c_void_p] +
+                         [c_int] * 6 + [c_void_p, c_size_t, c_void_p, c_void_p]),
     "nckv_delta_step": (c_int, [c_void_p] * 3 + [c_i64] * 3 + [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_i64, c_void_p, c_i64,
                                                             c_void_p, c_float, c_void_p, c_void_p] + [c_int] * 6 + [c_void_p]),
     "nckv_route_workspace_bytes": (c_size_t, [c_int] * 3),

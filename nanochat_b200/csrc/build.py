@@ -17,7 +17,7 @@ OUT = os.path.join(PKG, "libnckv.so")
 SOURCES = ["host.cu", "append.cu", "decode_attn.cu", "prefill_broadcast.cu", "lse_combine.cu",
            "prefill_attn.cu", "p2p_exchange.cu", "glue.cu", "flash_attn_bwd.cu", "host_step.cu",
            "recurrent.cu", "recurrent_f32.cu", "norm_mix.cu", "window_attn.cu", "hyper_norm.cu",
-           "gated_linear.cu", "delta.cu", "experts.cu", "experts_tc.cu"]
+           "gated_linear.cu", "delta.cu", "delta_chunk.cu", "experts.cu", "experts_tc.cu"]
 HEADERS = ["nckv_common.cuh", "vec_io.cuh", "tc05.cuh", "recurrent.cuh", "experts.cuh", os.path.join("..", "..", "include", "nckv.h")]
 
 

@@ -11,12 +11,13 @@
 //                         tile is the same for both operands and otherwise free.
 //   expert_plain_kernel   fp32, and sizes without 16-byte rows: 32 x 32 tiles on the fp32 pipe.
 // Many bf16 rows take the tensor-memory form in experts_tc.cu.
+#include <stdlib.h>
 #include "experts.cuh"
 
 namespace nckv {
 
 constexpr int RT_MAX_EXPERTS = 1024;
-constexpr int RT_ONE_CTA = 4096;  // (token, choice) pairs that one CTA sorts
+constexpr int RT_ONE_CTA = 2048;  // (token, choice) pairs that one CTA sorts
 
 struct RouteParams {
     const float *logits;   // (rows, E)
@@ -28,30 +29,36 @@ struct RouteParams {
     int rows, E, top;
 };
 
-// the best (logit, index) after (z_last, e_last) in the order "larger logit, then lower index"
-__device__ __forceinline__ void route_next(const float *z, int E, int lane, float &z_last, int &e_last) {
-    float best = -INFINITY;
-    int idx = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-        const float v = z[e];
-        const bool behind = v < z_last || (v == z_last && e > e_last);
-        if (behind && (v > best || (v == best && e < idx))) {
-            best = v;
-            idx = e;
-        }
-    }
+// A row's logits in the lanes of a warp, 32 NJ at most, as numbers whose unsigned order is theirs; 0: none, or taken.
+template <int NJ> struct RouteRow {
+    uint32_t key[NJ];
+    __device__ __forceinline__ void load(const float *z, int E, int lane) {
 #pragma unroll
-    for (int off = 16; off; off >>= 1) {
-        const float v = __shfl_xor_sync(0xffffffffu, best, off);
-        const int e = __shfl_xor_sync(0xffffffffu, idx, off);
-        if (v > best || (v == best && e < idx)) {
-            best = v;
-            idx = e;
+        for (int j = 0; j < NJ; ++j) {
+            const int e = lane + 32 * j;
+            const uint32_t bits = e < E ? __float_as_uint(z[e]) : 0u;
+            key[j] = e < E ? (bits & 0x80000000u ? ~bits : bits | 0x80000000u) : 0u;
         }
     }
-    z_last = best;
-    e_last = min(idx, E - 1);  // no candidate (not-a-number logits): any index that exists
-}
+    // the largest that is left (ties: the lowest index) and its logit
+    __device__ __forceinline__ int next(int E, int lane, float &z) {
+        uint32_t best = key[0];
+        int idx = lane;
+#pragma unroll
+        for (int j = 1; j < NJ; ++j)
+            if (key[j] > best) {
+                best = key[j];
+                idx = lane + 32 * j;
+            }
+        const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+        const int e = (int)__reduce_min_sync(0xffffffffu, best == top ? (unsigned)idx : 0x7fffffffu);
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+            if (e == lane + 32 * j) key[j] = 0u;
+        z = __uint_as_float(top & 0x80000000u ? top & 0x7fffffffu : ~top);
+        return min(e, E - 1);
+    }
+};
 
 // exclusive prefix sums of count[0 .. E) by the first warp; the total behind the last
 __device__ __forceinline__ void route_prefix(const int *count, int *first, int E) {
@@ -71,6 +78,7 @@ __device__ __forceinline__ void route_prefix(const int *count, int *first, int E
     if (threadIdx.x == 0) first[E] = carry;
 }
 
+template <int NJ>
 __global__ void __launch_bounds__(1024) route_kernel(const RouteParams p) {
     __shared__ int s_count[RT_MAX_EXPERTS], s_first[RT_MAX_EXPERTS + 1];
     __shared__ uint16_t s_choice[RT_ONE_CTA];
@@ -79,11 +87,11 @@ __global__ void __launch_bounds__(1024) route_kernel(const RouteParams p) {
     for (int e = tid; e < p.E; e += NT) s_count[e] = 0;
     __syncthreads();
     for (int row = tid >> 5; row < p.rows; row += NT >> 5) {
-        const float *z = p.logits + (long long)row * p.E;
-        float zl = INFINITY;
-        int el = -1;
+        RouteRow<NJ> z;
+        z.load(p.logits + (long long)row * p.E, p.E, lane);
         for (int j = 0; j < p.top; ++j) {
-            route_next(z, p.E, lane, zl, el);
+            float zl;
+            const int el = z.next(p.E, lane, zl);
             if (lane == 0) {
                 s_choice[row * p.top + j] = (uint16_t)el;
                 s_weight[row * p.top + j] = 1.f / (1.f + expf(-zl));
@@ -103,6 +111,7 @@ __global__ void __launch_bounds__(1024) route_kernel(const RouteParams p) {
     }
 }
 
+template <int NJ>
 __global__ void __launch_bounds__(256) route_pick_kernel(const RouteParams p) {
     __shared__ int s_count[RT_MAX_EXPERTS];
     const int tid = threadIdx.x, lane = tid & 31, R = p.rows * p.top;
@@ -110,11 +119,11 @@ __global__ void __launch_bounds__(256) route_pick_kernel(const RouteParams p) {
     for (int e = tid; e < p.E; e += 256) s_count[e] = 0;
     __syncthreads();
     for (int row = blockIdx.x * 8 + (tid >> 5); row < p.rows; row += gridDim.x * 8) {
-        const float *z = p.logits + (long long)row * p.E;
-        float zl = INFINITY;
-        int el = -1;
+        RouteRow<NJ> z;
+        z.load(p.logits + (long long)row * p.E, p.E, lane);
         for (int j = 0; j < p.top; ++j) {
-            route_next(z, p.E, lane, zl, el);
+            float zl;
+            const int el = z.next(p.E, lane, zl);
             if (lane == 0) {
                 p.choice[row * p.top + j] = el;
                 p.weight[row * p.top + j] = 1.f / (1.f + expf(-zl));
@@ -298,7 +307,10 @@ static cudaError_t expert_plain(const ExpertParams &p, bool up, cudaStream_t s) 
 }
 
 // pairs above which the tensor-memory form is used
-static int expert_many(int E) { return 48 * E > 512 ? 48 * E : 512; }
+static int expert_many(int E) {
+    if (const char *v = getenv("NCKV_DEV_MANY")) return atoi(v);
+    return 48 * E > 512 ? 48 * E : 512;
+}
 
 }  // namespace nckv
 
@@ -326,8 +338,11 @@ int nckv_route(const float *logits, int32_t *offsets, int32_t *slot, float *scal
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int R = rows * top;
     if (R <= RT_ONE_CTA) {
-        const int warps = rows < 32 ? rows : 32;
-        route_kernel<<<1, warps * 32, 0, s>>>(p);
+        const int threads = 32 * (rows < 4 ? 4 : (rows < 32 ? rows : 32));
+        if (E <= 32) route_kernel<1><<<1, threads, 0, s>>>(p);
+        else if (E <= 64) route_kernel<2><<<1, threads, 0, s>>>(p);
+        else if (E <= 256) route_kernel<8><<<1, threads, 0, s>>>(p);
+        else route_kernel<32><<<1, threads, 0, s>>>(p);
         NCKV_CUDA_CHECK(cudaGetLastError());
         return NCKV_OK;
     }
@@ -340,7 +355,10 @@ int nckv_route(const float *logits, int32_t *offsets, int32_t *slot, float *scal
     NCKV_CUDA_CHECK(cudaMemsetAsync(p.choice + R, 0, sizeof(int32_t) * 2 * E, s));
     int grid = (rows + 7) / 8;
     if (grid > 4 * sm_count()) grid = 4 * sm_count();
-    route_pick_kernel<<<grid, 256, 0, s>>>(p);
+    if (E <= 32) route_pick_kernel<1><<<grid, 256, 0, s>>>(p);
+    else if (E <= 64) route_pick_kernel<2><<<grid, 256, 0, s>>>(p);
+    else if (E <= 256) route_pick_kernel<8><<<grid, 256, 0, s>>>(p);
+    else route_pick_kernel<32><<<grid, 256, 0, s>>>(p);
     NCKV_CUDA_CHECK(cudaGetLastError());
     const int per = (R + sm_count() - 1) / sm_count() < 1024 ? 1024 : (R + sm_count() - 1) / sm_count();
     route_place_kernel<<<(R + per - 1) / per, 256, 0, s>>>(p, per);

@@ -3,15 +3,16 @@
 // Persistent CTAs, one per SM, walk over the tiles of all experts: 128 of an expert's sorted positions by BN
 // weight rows (UP: BN / 2 gate and the BN / 2 up rows of the same channels, so that a thread holds both
 // factors of an output).  A tile's K runs in steps of 64 through a ring in shared memory (128-byte
-// swizzle).  Four roles, connected by mbarriers:
-//   warp 0      moves the operands by TMA.  UP: the tokens of a tile lie anywhere in h; every lane fetches
-//               four of the 128 rows per step with one gather (tile::gather4), so h is never copied into
-//               sorted order.  Otherwise the positions are rows of act, one plain copy.
+// swizzle).  Roles, connected by mbarriers:
+//   warp 0      moves the weights, and without UP the positions (rows of act), by TMA
+//   warps 6-9   UP: the tokens of a tile lie anywhere in h; these warps fetch them with 16-byte asynchronous copies
+//               into the place the swizzle gives them, so h is never copied into sorted order (a gather by
+//               TMA, four rows per instruction, was three times slower than the products).
 //   warp 1      one thread issues the products into one of two accumulators
 //   warps 2-5   one thread per position reads the other accumulator, applies the router's weight and the
 //               activation (UP) or finds the pair's place (down), and stores
 // Tiles of one expert are consecutive, positions fastest: the CTAs that run side by side share weights and rows
-// in L2.  Positions behind an expert's last repeat it and are not stored.  Every wait is bounded; one that
+// in L2.  What stands in a tile behind an expert's last position is not stored.  Every wait is bounded; one that
 // runs out sets NCKV_ST_TIMEOUT, the roles stop, copies in flight are waited for and tensor memory is freed.
 #include "experts.cuh"
 #include "tc05.cuh"
@@ -19,7 +20,7 @@
 namespace nckv {
 
 constexpr int ET_M = 128, ET_K = 64;
-constexpr int ET_THREADS = 192;
+constexpr int ET_THREADS = 192, ET_GATHER = 128;  // UP has ET_GATHER more
 constexpr int ET_MAX_EXPERTS = 1024;
 constexpr int ET_A_BYTES = ET_M * ET_K * 2;
 
@@ -45,7 +46,7 @@ struct EtCursor {
 };
 
 template <bool UP, int BN>
-__global__ void __launch_bounds__(ET_THREADS, 1)
+__global__ void __launch_bounds__(ET_THREADS + (UP ? ET_GATHER : 0), 1)
 experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, const ExpertParams p) {
     using Shape = EtShape<BN>;
     constexpr int STAGES = Shape::STAGES;
@@ -85,7 +86,7 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
         prefetch_tensormap(&map_a);
         prefetch_tensormap(&map_w);
         for (int i = 0; i < STAGES; ++i) {
-            mbar_init(&bar_full[i], 1);
+            mbar_init(&bar_full[i], UP ? 1 + ET_GATHER / 32 : 1);
             mbar_init(&bar_free[i], 1);
         }
         for (int i = 0; i < 2; ++i) {
@@ -120,11 +121,6 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
         bool ok = true;
         for (int idx = blockIdx.x; idx < total && ok; idx += gridDim.x) {
             if (!cur.seek(s_first, p, n_tiles, idx)) break;
-            int r[4] = {0, 0, 0, 0};
-            if (UP) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) r[i] = p.slot[min(cur.m0 + lane * 4 + i, cur.m_hi - 1)] / p.top;
-            }
             for (int ks = 0; ks < k_steps; ++ks, ++fill) {
                 const uint32_t st = fill % STAGES, round = fill / STAGES;
                 if (round > 0 && !warp_wait(&bar_free[st], (round - 1) & 1u)) {
@@ -132,14 +128,15 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
                     break;
                 }
                 uint8_t *a = smem + st * Shape::STAGE, *b = a + ET_A_BYTES;
-                if (lane == 0) mbar_arrive_expect_tx(&bar_full[st], Shape::STAGE);
-                __syncwarp();
-                if (UP) {
-                    tma_gather4(a + lane * 512, &map_a, &bar_full[st], ks * ET_K, r[0], r[1], r[2], r[3]);
-                    if (lane < 2) tma_load_4d(b + lane * (Shape::B_BYTES / 2), &map_w, &bar_full[st], ks * ET_K, cur.n * (BN / 2), lane, cur.e);
-                } else if (lane == 0) {
-                    tma_load_2d(a, &map_a, &bar_full[st], ks * ET_K, cur.m0);
-                    tma_load_4d(b, &map_w, &bar_full[st], ks * ET_K, cur.n * BN, 0, cur.e);
+                if (lane == 0) {
+                    mbar_arrive_expect_tx(&bar_full[st], UP ? Shape::B_BYTES : Shape::STAGE);
+                    if (UP) {
+                        tma_load_4d(b, &map_w, &bar_full[st], ks * ET_K, cur.n * (BN / 2), 0, cur.e);
+                        tma_load_4d(b + Shape::B_BYTES / 2, &map_w, &bar_full[st], ks * ET_K, cur.n * (BN / 2), 1, cur.e);
+                    } else {
+                        tma_load_2d(a, &map_a, &bar_full[st], ks * ET_K, cur.m0);
+                        tma_load_4d(b, &map_w, &bar_full[st], ks * ET_K, cur.n * BN, 0, cur.e);
+                    }
                 }
             }
         }
@@ -184,6 +181,55 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
             }
             if (!ok) timed_out();
         }
+        __syncwarp();
+    } else if (UP && warp >= 6) {
+        // =============== tokens =====================================================================
+        // 8 threads fetch the 128 bytes a token has in a step; a thread serves 8 tokens.  A step is handed over
+        // once the LAG steps behind it have been asked for.
+        constexpr int LAG = STAGES - 1;
+        const int pt = tid - ET_THREADS, chunk = pt & 7, r0 = pt >> 3;
+        uint32_t fill = 0;
+        bool ok = true;
+        auto hand_over = [&](uint32_t f) {
+            fence_proxy_async_smem();  // this thread's copies, before the products read them
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&bar_full[f % STAGES]);
+        };
+        for (int idx = blockIdx.x; idx < total && ok; idx += gridDim.x) {
+            if (!cur.seek(s_first, p, n_tiles, idx)) break;
+            const __nv_bfloat16 *src[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int m = cur.m0 + r0 + 16 * i;  // nobody reads the results of rows behind the expert's last
+                src[i] = m < cur.m_hi ? static_cast<const __nv_bfloat16 *>(p.a) + (long long)(p.slot[m] / p.top) * p.K + chunk * 8 : nullptr;
+            }
+            for (int ks = 0; ks < k_steps; ++ks, ++fill) {
+                const uint32_t st = fill % STAGES, round = fill / STAGES;
+                if (round > 0 && !warp_wait(&bar_free[st], (round - 1) & 1u)) {
+                    ok = false;
+                    break;
+                }
+                const uint32_t base = smem_u32(smem + st * Shape::STAGE);
+                const int bytes = ks * ET_K + chunk * 8 < p.K ? 16 : 0;  // zeros behind the last channel
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int r = r0 + 16 * i;
+                    if (src[i])
+                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(base + r * 128 + ((chunk ^ (r & 7)) << 4)),
+                                     "l"(bytes ? src[i] + ks * ET_K : src[i]), "r"(bytes)
+                                     : "memory");
+                }
+                asm volatile("cp.async.commit_group;" ::: "memory");
+                if (fill >= (uint32_t)LAG) {
+                    asm volatile("cp.async.wait_group %0;" ::"n"(LAG) : "memory");
+                    hand_over(fill - LAG);
+                }
+            }
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        if (ok)
+            for (uint32_t f = fill > (uint32_t)LAG ? fill - LAG : 0; f < fill; ++f) hand_over(f);
+        else if (lane == 0 && *abort_flag == 0) timed_out();
         __syncwarp();
     } else {
         // =============== results ====================================================================
@@ -246,14 +292,10 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
 template <bool UP, int BN>
 static cudaError_t et_launch(const ExpertParams &p, cudaStream_t s, int *rc) {
     CUtensorMap ma, mw;
-    if (UP) {
-        const int64_t dims[2] = {p.K, p.R / p.top}, strides[1] = {p.K};
-        const int box[2] = {ET_K, 1};  // the gather fetches its rows one by one
-        *rc = make_tensor_map(&ma, p.a, 2, dims, strides, box);
-    } else {
-        const int64_t dims[2] = {p.K, p.R}, strides[1] = {p.K};
+    {
+        const int64_t dims[2] = {p.K, UP ? p.R / p.top : p.R}, strides[1] = {p.K};
         const int box[2] = {ET_K, ET_M};
-        *rc = make_tensor_map(&ma, p.a, 2, dims, strides, box);
+        *rc = make_tensor_map(&ma, p.a, 2, dims, strides, box);  // not used by UP
     }
     if (*rc != NCKV_OK) return cudaSuccess;
     const int64_t N = p.N, K = p.K, halves = UP ? 2 : 1;
@@ -265,7 +307,7 @@ static cudaError_t et_launch(const ExpertParams &p, cudaStream_t s, int *rc) {
     if (e != cudaSuccess) return e;
     const long long tiles = ((long long)p.R / ET_M + p.E) * ((p.N + BN / halves - 1) / (BN / halves));
     const int grid = tiles < sm_count() ? (int)tiles : sm_count();
-    experts_tc_kernel<UP, BN><<<grid, ET_THREADS, EtShape<BN>::SMEM, s>>>(ma, mw, p);
+    experts_tc_kernel<UP, BN><<<grid, ET_THREADS + (UP ? ET_GATHER : 0), EtShape<BN>::SMEM, s>>>(ma, mw, p);
     return cudaGetLastError();
 }
 

@@ -2,15 +2,14 @@
 //
 //   short_conv_kernel   out_t = act(b + sum_j taps[j] (x_(t - K + 1 + j) + b_in)), per channel, zeros before the
 //                       start of a sequence; the last K - 1 inputs of every row are carried in fp32.  A
-//                       thread slides over a run of tokens of 4 (or 1) channels with the inputs in registers.
+//                       thread takes a run of tokens of 4 (or 1) channels, all inputs loaded together.
 //   conv_carry_kernel   the carried inputs after a call of more than one run
 //   gated_scan_kernel   S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with log a_t = -rate r_t and the gates
-//                       r, i = sigmoid(logits + bias); out_t = S_t * gelu_tanh(y_t + b_y).  A CTA owns L
-//                       channels of one row; its warps (or half-warps) take SC_TOKENS consecutive tokens each,
-//                       find their own decay product and contribution, chain them through shared memory and
-//                       run through their tokens again from the right initial state (operands stay in
-//                       registers, so global memory is read once).
-//   gated_scan_step_kernel   the same for few tokens: a thread per channel, one token after the other.
+//                       r, i = sigmoid(logits + bias); out_t = S_t * gelu_tanh(y_t + b_y).  A thread per channel
+//                       and segment.  Prompts are cut into segments that run side by side: a first pass
+//                       finds each segment's decay product and own contribution, gated_join_kernel chains
+//                       them, a second pass runs all segments from their initial states.  How the tokens
+//                       are cut changes results at fp32 rounding level only.
 #include "vec_io.cuh"
 
 namespace nckv {
@@ -18,7 +17,7 @@ namespace nckv {
 // ------------------------------------------------------------------------------------------------
 // short causal convolution
 // ------------------------------------------------------------------------------------------------
-constexpr int CONV_RUN = 16;
+constexpr int CONV_RUN = 8;
 constexpr int CONV_MAX_TAPS = 16;
 
 struct ShortConvParams {
@@ -28,86 +27,98 @@ struct ShortConvParams {
     const float *in_bias, *bias;  // (C) or null
     float *carry;           // (B, K - 1, C)
     void *out;              // (B * T, C) T
-    int B, T, C, K, run, act;
+    int B, T, C, K, act;
 };
 
-template <typename T, int V, int KK>
+// KK: taps of the padded filter (the first KK - K are zero).  RUN tokens per thread, their inputs loaded together.
+template <typename T, int V, int KK, int RUN>
 __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p) {
     const int c = (blockIdx.x * 128 + threadIdx.x) * V, b = blockIdx.z;
     if (c >= p.C) return;
-    const int t0 = blockIdx.y * p.run, t1 = min(p.T, t0 + p.run);
-    const int K = p.K, lack = KK - K;  // the first `lack` taps of the padded filter are zero
-    float w[KK][V], win[KK][V], bi[V], bo[V];
+    const int t0 = blockIdx.y * RUN, K = p.K, lack = KK - K;
+    const T *x = static_cast<const T *>(p.x) + (long long)b * p.T * p.x_stride + c;
+    float *carry = p.carry + (long long)b * (K - 1) * p.C + c;
+    float in[RUN + KK - 1][V], bi[V], bo[V];  // in[j]: input of token t0 - (KK - 1) + j
 #pragma unroll
     for (int e = 0; e < V; ++e) bi[e] = bo[e] = 0.f;
     if (p.in_bias) get_v(p.in_bias + c, bi);
     if (p.bias) get_v(p.bias + c, bo);
-    const T *x = static_cast<const T *>(p.x) + (long long)b * p.T * p.x_stride + c;
-    float *carry = p.carry + (long long)b * (K - 1) * p.C + c;
-    auto input = [&](int t, float (&o)[V]) {  // input of token t of this call; before it: what is carried
-        if (t >= 0) {
-            get_v(x + t * p.x_stride, o);
 #pragma unroll
-            for (int e = 0; e < V; ++e) o[e] += bi[e];
-        } else {
-            get_v(carry + (long long)(K - 1 + t) * p.C, o);
+    for (int j = 0; j < RUN + KK - 1; ++j) {
+        const int t = t0 - (KK - 1) + j;
+#pragma unroll
+        for (int e = 0; e < V; ++e) in[j][e] = 0.f;
+        if (j < lack || t >= p.T) continue;
+        if (t >= 0) get_v(x + t * p.x_stride, in[j]);
+        else get_v(carry + (long long)(K - 1 + t) * p.C, in[j]);  // what is carried has its bias already
+    }
+#pragma unroll
+    for (int j = 0; j < RUN + KK - 1; ++j)
+        if (t0 - (KK - 1) + j >= 0) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) in[j][e] += bi[e];
         }
-    };
+    float w[KK][V];
 #pragma unroll
     for (int j = 0; j < KK; ++j) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) w[j][e] = win[j][e] = 0.f;
+        for (int e = 0; e < V; ++e) w[j][e] = 0.f;
         if (j >= lack) get_v(p.taps + (long long)(j - lack) * p.C + c, w[j]);
-        if (j >= lack && j < KK - 1) input(t0 - (KK - 1) + j, win[j]);
     }
-    for (int t = t0; t < t1; ++t) {
-        input(t, win[KK - 1]);
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+        if (t0 + i >= p.T) break;
         float o[V];
 #pragma unroll
         for (int e = 0; e < V; ++e) {
             o[e] = bo[e];
 #pragma unroll
-            for (int j = 0; j < KK; ++j) o[e] = fmaf(w[j][e], win[j][e], o[e]);
+            for (int j = 0; j < KK; ++j) o[e] = fmaf(w[j][e], in[i + j][e], o[e]);
             if (p.act) o[e] = Fn<T>::silu(o[e]);
         }
-        put_v(static_cast<T *>(p.out) + ((long long)b * p.T + t) * p.C + c, o);
-#pragma unroll
-        for (int j = 0; j < KK - 1; ++j)
-#pragma unroll
-            for (int e = 0; e < V; ++e) win[j][e] = win[j + 1][e];
+        put_v(static_cast<T *>(p.out) + ((long long)b * p.T + t0 + i) * p.C + c, o);
     }
-    if (p.run >= p.T) {  // the only run of its row: nobody else reads the carried inputs
+    if (gridDim.y == 1) {  // the only run of its row: nobody else reads the carried inputs
 #pragma unroll
-        for (int j = 0; j < KK - 1; ++j)
-            if (j >= lack) put_v(carry + (long long)(j - lack) * p.C, win[j]);
+        for (int j = 1; j < RUN + KK - 1; ++j) {
+            const int keep = j - lack - p.T;  // token t0 - (KK - 1) + j is number `keep` of the K - 1 to carry
+            if (keep >= 0 && keep < K - 1) put_v(carry + (long long)keep * p.C, in[j]);
+        }
     }
 }
 
-// after a call of T >= K - 1 tokens
+// the carried inputs after a call: the last K - 1 of those carried before and the call's own
 template <typename T>
 __global__ void __launch_bounds__(256) conv_carry_kernel(const ShortConvParams p) {
-    const int c = blockIdx.x * 256 + threadIdx.x, j = blockIdx.y, b = blockIdx.z;
+    const int c = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y;
     if (c >= p.C) return;
-    const long long t = (long long)b * p.T + p.T - (p.K - 1) + j;
-    p.carry[((long long)b * (p.K - 1) + j) * p.C + c] =
-        to_f(static_cast<const T *>(p.x)[t * p.x_stride + c]) + (p.in_bias ? p.in_bias[c] : 0.f);
+    const float bias = p.in_bias ? p.in_bias[c] : 0.f;
+    float *carry = p.carry + (long long)b * (p.K - 1) * p.C + c;
+    for (int j = 0; j < p.K - 1; ++j) {  // reads run ahead of writes
+        const int t = p.T - (p.K - 1) + j;
+        carry[(long long)j * p.C] = t >= 0 ? to_f(static_cast<const T *>(p.x)[((long long)b * p.T + t) * p.x_stride + c]) + bias
+                                           : carry[(long long)(j + p.T) * p.C];
+    }
+}
+
+template <typename T, int V, int RUN>
+static cudaError_t conv_run(const ShortConvParams &p, cudaStream_t s) {
+    const dim3 grid((p.C + 128 * V - 1) / (128 * V), (p.T + RUN - 1) / RUN, p.B);
+    if (p.K <= 2) short_conv_kernel<T, V, 2, RUN><<<grid, 128, 0, s>>>(p);
+    else if (p.K <= 4) short_conv_kernel<T, V, 4, RUN><<<grid, 128, 0, s>>>(p);
+    else if (p.K <= 8) short_conv_kernel<T, V, 8, RUN><<<grid, 128, 0, s>>>(p);
+    else short_conv_kernel<T, V, CONV_MAX_TAPS, RUN><<<grid, 128, 0, s>>>(p);
+    return cudaGetLastError();
 }
 
 template <typename T, int V>
-static cudaError_t conv_launch(ShortConvParams p, cudaStream_t s) {
-    // runs long enough to make the K - 1 inputs read again cheap; short calls in one run
-    p.run = p.T <= CONV_RUN ? p.T : CONV_RUN;
-    const dim3 grid((p.C + 128 * V - 1) / (128 * V), (p.T + p.run - 1) / p.run, p.B);
-    if (p.K <= 2) short_conv_kernel<T, V, 2><<<grid, 128, 0, s>>>(p);
-    else if (p.K <= 4) short_conv_kernel<T, V, 4><<<grid, 128, 0, s>>>(p);
-    else if (p.K <= 8) short_conv_kernel<T, V, 8><<<grid, 128, 0, s>>>(p);
-    else short_conv_kernel<T, V, CONV_MAX_TAPS><<<grid, 128, 0, s>>>(p);
-    cudaError_t e = cudaGetLastError();
-    if (e != cudaSuccess || p.run >= p.T || p.K == 1) return e;
-    conv_carry_kernel<T><<<dim3((p.C + 255) / 256, p.K - 1, p.B), 256, 0, s>>>(p);  // T > CONV_RUN >= K here
+static cudaError_t conv_launch(const ShortConvParams &p, cudaStream_t s) {
+    if (p.T == 1) return conv_run<T, V, 1>(p, s);
+    const cudaError_t e = conv_run<T, V, CONV_RUN>(p, s);
+    if (e != cudaSuccess || p.T <= CONV_RUN || p.K == 1) return e;
+    conv_carry_kernel<T><<<dim3((p.C + 255) / 256, p.B), 256, 0, s>>>(p);
     return cudaGetLastError();
 }
-static_assert(CONV_RUN >= CONV_MAX_TAPS, "the carried inputs of a longer call are all its own");
 
 // ------------------------------------------------------------------------------------------------
 // real-gated linear recurrence
@@ -121,103 +132,108 @@ struct GatedScanParams {
     const float *rate;       // (C), >= 0
     float *state;            // (B, C)
     void *out;               // (B * T, C) T
-    int B, T, C, n;
+    float *parts;            // (B, n_seg, 2, C): own contribution, then initial state; decay product
+    int B, T, C, n, n_seg;
 };
 
-// decay and drive of one token
-template <typename T>
-__device__ __forceinline__ void gated_terms(float zr, float zi, float rate, float u, float &a, float &d) {
-    const float la = -rate * Fn<T>::sigmoid(zr);
-    a = Fn<T>::exp(la);
-    d = sqrtf(-expm1f(2.f * la)) * Fn<T>::sigmoid(zi) * u;
+// decay and drive of one token; sqrt(1 - a^2) from log a, which keeps its digits where a is close to 1
+template <typename T> __device__ __forceinline__ void gated_terms(float zr, float zi, float rate, float u, float &a, float &d);
+template <> __device__ __forceinline__ void gated_terms<float>(float zr, float zi, float rate, float u, float &a, float &d) {
+    const float la = -rate * Fn<float>::sigmoid(zr);
+    a = expf(la);
+    d = sqrtf(-expm1f(2.f * la)) * Fn<float>::sigmoid(zi) * u;
+}
+template <> __device__ __forceinline__ void gated_terms<__nv_bfloat16>(float zr, float zi, float rate, float u, float &a, float &d) {
+    const float la = -rate * Fn<__nv_bfloat16>::sigmoid(zr), x = -2.f * la;
+    a = __expf(la);
+    // 1 - e^-x: its series where the difference would cancel (the first term left out is x^6 / 720)
+    const float small = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, -1.f / 24.f), 1.f / 6.f), -0.5f), 1.f);
+    const float y = x < 0.125f ? small : fmaf(-a, a, 1.f);
+    d = (y > 0.f ? y * rsqrtf(y) : 0.f) * Fn<__nv_bfloat16>::sigmoid(zi) * u;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(128) gated_scan_step_kernel(const GatedScanParams p) {
-    const int c = blockIdx.x * 128 + threadIdx.x, b = blockIdx.y;
+constexpr int SC_SEG = 32;   // tokens per segment
+constexpr int SC_AHEAD = 8;  // tokens whose operands are loaded together
+
+// SCAN: 0 all tokens of a row from its state (few tokens), 1 a segment's decay product and own contribution,
+// 2 a segment's outputs from its initial state
+template <typename T, int SCAN>
+__global__ void __launch_bounds__(128) gated_scan_kernel(const GatedScanParams p) {
+    const int c = blockIdx.x * 128 + threadIdx.x, b = blockIdx.z, seg = blockIdx.y;
     if (c >= p.C) return;
-    const int blk = c / p.n, j = c - blk * p.n;
-    const float br = p.gate_bias[c], bi = p.gate_bias[p.C + c], by = p.y_bias[c], rate = p.rate[c];
-    float S = p.state[(long long)b * p.C + c];
-    for (int t = 0; t < p.T; ++t) {
-        const long long row = (long long)b * p.T + t;
-        const float *g = p.gates + ((long long)blk * p.B * p.T + row) * 2 * p.n + j;
-        float a, d;
-        gated_terms<T>(g[0] + br, g[p.n] + bi, rate, to_f(static_cast<const T *>(p.u)[row * p.u_stride + c]), a, d);
-        S = fmaf(a, S, d);
-        put(static_cast<T *>(p.out) + row * p.C + c, S * gelu_tanh<T>(to_f(static_cast<const T *>(p.y)[row * p.y_stride + c]) + by));
-    }
-    p.state[(long long)b * p.C + c] = S;
-}
-
-constexpr int SC_TOKENS = 16;   // consecutive tokens a thread holds
-constexpr int SC_THREADS = 256;
-
-// L: channels per CTA; SC_THREADS / L groups of tokens
-template <typename T, int L>
-__global__ void __launch_bounds__(SC_THREADS) gated_scan_kernel(const GatedScanParams p) {
-    constexpr int NG = SC_THREADS / L, CHUNK = NG * SC_TOKENS;
-    __shared__ float s_prod[2][NG][L], s_end[2][NG][L];
-    const int lane = threadIdx.x % L, grp = threadIdx.x / L, b = blockIdx.y;
-    const int c_raw = blockIdx.x * L + lane, c = min(c_raw, p.C - 1);  // spare lanes repeat the last channel
-    const bool have = c_raw < p.C;
     const int blk = c / p.n, j = c - blk * p.n;
     const float br = p.gate_bias[c], bi = p.gate_bias[p.C + c], by = p.y_bias[c], rate = p.rate[c];
     const long long row0 = (long long)b * p.T;
     const T *u = static_cast<const T *>(p.u) + row0 * p.u_stride + c, *y = static_cast<const T *>(p.y) + row0 * p.y_stride + c;
     const float *g = p.gates + ((long long)blk * p.B * p.T + row0) * 2 * p.n + j;
     T *out = static_cast<T *>(p.out) + row0 * p.C + c;
-    float S = p.state[(long long)b * p.C + c];
-    int parity = 0;
-    for (int t0 = 0; t0 < p.T; t0 += CHUNK, parity ^= 1) {
-        const int t = t0 + grp * SC_TOKENS;
-        float a[SC_TOKENS], d[SC_TOKENS], yv[SC_TOKENS];
+    float *part = p.parts + ((long long)b * p.n_seg + seg) * 2 * p.C + c;
+    const int t_begin = SCAN ? seg * SC_SEG : 0, t_end = SCAN ? min(p.T, t_begin + SC_SEG) : p.T;
+    float S = SCAN == 0 ? p.state[(long long)b * p.C + c] : (SCAN == 2 ? part[0] : 0.f), prod = 1.f;
+    for (int t0 = t_begin; t0 < t_end; t0 += SC_AHEAD) {
+        float zr[SC_AHEAD], zi[SC_AHEAD];
+        T uu[SC_AHEAD], yy[SC_AHEAD];
 #pragma unroll
-        for (int i = 0; i < SC_TOKENS; ++i) {  // all loads first
-            const long long r = min(t + i, p.T - 1);
-            a[i] = g[r * 2 * p.n];
-            d[i] = g[r * 2 * p.n + p.n];
-            yv[i] = to_f(y[r * p.y_stride]);
-        }
-        float prod = 1.f, end = 0.f;
-#pragma unroll
-        for (int i = 0; i < SC_TOKENS; ++i) {
-            const long long r = min(t + i, p.T - 1);
-            float an, dn;
-            gated_terms<T>(a[i] + br, d[i] + bi, rate, to_f(u[r * p.u_stride]), an, dn);
-            const bool in = t + i < p.T;
-            a[i] = in ? an : 1.f;
-            d[i] = in ? dn : 0.f;
-            prod *= a[i];
-            end = fmaf(a[i], end, d[i]);
-        }
-        s_prod[parity][grp][lane] = prod;
-        s_end[parity][grp][lane] = end;
-        __syncthreads();  // the other buffer is free again once all have passed here
-        float mine = S;
-#pragma unroll
-        for (int q = 0; q < NG; ++q) {
-            if (q == grp) mine = S;
-            S = fmaf(s_prod[parity][q][lane], S, s_end[parity][q][lane]);
+        for (int i = 0; i < SC_AHEAD; ++i) {
+            const long long t = min(t0 + i, t_end - 1);
+            zr[i] = g[t * 2 * p.n];
+            zi[i] = g[t * 2 * p.n + p.n];
+            uu[i] = u[t * p.u_stride];
+            if (SCAN != 1) yy[i] = y[t * p.y_stride];
         }
 #pragma unroll
-        for (int i = 0; i < SC_TOKENS; ++i) {
-            mine = fmaf(a[i], mine, d[i]);
-            if (have && t + i < p.T) put(out + (long long)(t + i) * p.C, mine * gelu_tanh<T>(yv[i] + by));
+        for (int i = 0; i < SC_AHEAD; ++i) {
+            if (t0 + i >= t_end) break;
+            float a, d;
+            gated_terms<T>(zr[i] + br, zi[i] + bi, rate, to_f(uu[i]), a, d);
+            S = fmaf(a, S, d);
+            if (SCAN == 1) prod *= a;
+            else put(out + (long long)(t0 + i) * p.C, S * gelu_tanh<T>(to_f(yy[i]) + by));
         }
     }
-    if (have && grp == 0) p.state[(long long)b * p.C + c] = S;
+    if (SCAN == 0) p.state[(long long)b * p.C + c] = S;
+    if (SCAN == 1) {
+        part[0] = S;
+        part[p.C] = prod;
+    }
 }
+
+// every segment's initial state in place of its own contribution, and the row's state after the last
+__global__ void __launch_bounds__(64) gated_join_kernel(const GatedScanParams p) {
+    const int c = blockIdx.x * 64 + threadIdx.x, b = blockIdx.y;
+    if (c >= p.C) return;
+    float *part = p.parts + (long long)b * p.n_seg * 2 * p.C + c;
+    float S = p.state[(long long)b * p.C + c];
+    for (int s0 = 0; s0 < p.n_seg; s0 += 16) {
+        float own[16], prod[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            const long long at = (long long)min(s0 + i, p.n_seg - 1) * 2 * p.C;
+            own[i] = part[at];
+            prod[i] = part[at + p.C];
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            if (s0 + i >= p.n_seg) break;
+            part[(long long)(s0 + i) * 2 * p.C] = S;
+            S = fmaf(prod[i], S, own[i]);
+        }
+    }
+    p.state[(long long)b * p.C + c] = S;
+}
+
+static int scan_segments(int T) { return T <= SC_SEG ? 0 : (T + SC_SEG - 1) / SC_SEG; }
 
 template <typename T>
 static cudaError_t scan_launch(const GatedScanParams &p, cudaStream_t s) {
-    if (p.T <= SC_TOKENS) {
-        gated_scan_step_kernel<T><<<dim3((p.C + 127) / 128, p.B), 128, 0, s>>>(p);
-    } else if ((long long)p.B * ((p.C + 31) / 32) >= 2 * sm_count()) {
-        gated_scan_kernel<T, 32><<<dim3((p.C + 31) / 32, p.B), SC_THREADS, 0, s>>>(p);
-    } else {
-        gated_scan_kernel<T, 16><<<dim3((p.C + 15) / 16, p.B), SC_THREADS, 0, s>>>(p);
+    const unsigned cols = (p.C + 127) / 128;
+    if (p.n_seg == 0) {
+        gated_scan_kernel<T, 0><<<dim3(cols, 1, p.B), 128, 0, s>>>(p);
+        return cudaGetLastError();
     }
+    gated_scan_kernel<T, 1><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
+    gated_join_kernel<<<dim3((p.C + 63) / 64, p.B), 64, 0, s>>>(p);
+    gated_scan_kernel<T, 2><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
     return cudaGetLastError();
 }
 
@@ -232,7 +248,7 @@ int nckv_short_conv(const void *x, int64_t x_stride, const float *taps, const fl
         set_error("short_conv: null pointer argument");
         return NCKV_E_ARG;
     }
-    if (B <= 0 || T <= 0 || C <= 0 || K <= 0 || B > 65535 || (T + CONV_RUN - 1) / CONV_RUN > 65535) {
+    if (B <= 0 || T <= 0 || C <= 0 || K <= 0 || B > 65535 || T > 65535 * CONV_RUN) {
         set_error("short_conv: size out of range (B=%d T=%d C=%d K=%d)", B, T, C, K);
         return NCKV_E_ARG;
     }
@@ -242,7 +258,7 @@ int nckv_short_conv(const void *x, int64_t x_stride, const float *taps, const fl
     }
     ShortConvParams p;
     p.x = x; p.x_stride = x_stride; p.taps = taps; p.in_bias = in_bias; p.bias = bias; p.carry = carry; p.out = out;
-    p.B = B; p.T = T; p.C = C; p.K = K; p.run = T; p.act = act;
+    p.B = B; p.T = T; p.C = C; p.K = K; p.act = act;
     const uintptr_t elem = f32 ? 4 : 2;
     const uintptr_t a32 = (uintptr_t)taps | (uintptr_t)in_bias | (uintptr_t)bias | (uintptr_t)carry;
     const uintptr_t at = (uintptr_t)x | (uintptr_t)out | (uintptr_t)x_stride * elem;
@@ -255,9 +271,14 @@ int nckv_short_conv(const void *x, int64_t x_stride, const float *taps, const fl
     return NCKV_OK;
 }
 
+size_t nckv_gated_scan_workspace_bytes(int B, int T, int C) {
+    if (B <= 0 || T <= 0 || C <= 0) return 0;
+    return sizeof(float) * 2 * (size_t)B * nckv::scan_segments(T) * C;
+}
+
 int nckv_gated_scan(const void *u, int64_t u_stride, const void *y, int64_t y_stride, const float *gates, const float *gate_bias,
                     const float *y_bias, const float *rate, float *state, void *out, int B, int T, int C, int blocks, int f32,
-                    void *stream) {
+                    void *workspace, size_t workspace_bytes, void *stream) {
     using namespace nckv;
     if (!u || !y || !gates || !gate_bias || !y_bias || !rate || !state || !out) {
         set_error("gated_scan: null pointer argument");
@@ -267,10 +288,15 @@ int nckv_gated_scan(const void *u, int64_t u_stride, const void *y, int64_t y_st
         set_error("gated_scan: size out of range (B=%d T=%d C=%d blocks=%d)", B, T, C, blocks);
         return NCKV_E_ARG;
     }
+    if (scan_segments(T) > 65535 || (scan_segments(T) && (!workspace || workspace_bytes < nckv_gated_scan_workspace_bytes(B, T, C)))) {
+        set_error("gated_scan: workspace of %zu bytes given, %zu needed", workspace_bytes, nckv_gated_scan_workspace_bytes(B, T, C));
+        return NCKV_E_CAPACITY;
+    }
     GatedScanParams p;
     p.u = u; p.y = y; p.u_stride = u_stride; p.y_stride = y_stride;
     p.gates = gates; p.gate_bias = gate_bias; p.y_bias = y_bias; p.rate = rate; p.state = state; p.out = out;
-    p.B = B; p.T = T; p.C = C; p.n = C / blocks;
+    p.parts = static_cast<float *>(workspace);
+    p.B = B; p.T = T; p.C = C; p.n = C / blocks; p.n_seg = scan_segments(T);
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     NCKV_CUDA_CHECK(f32 ? scan_launch<float>(p, s) : scan_launch<__nv_bfloat16>(p, s));
     return NCKV_OK;

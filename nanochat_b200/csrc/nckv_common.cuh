@@ -189,15 +189,6 @@ __device__ __forceinline__ void tma_load_2d(void *smem_dst, const CUtensorMap *m
         "l"(map), "r"(c0), "r"(c1), "r"(smem_u32(bar))
         : "memory");
 }
-// Four rows of a 2-D map whose box is one row high, one after the other in shared memory.
-__device__ __forceinline__ void tma_gather4(void *smem_dst, const CUtensorMap *map, uint64_t *bar, int c0, int r0, int r1,
-                                            int r2, int r3) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes"
-        " [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(smem_u32(smem_dst)),
-        "l"(map), "r"(c0), "r"(r0), "r"(r1), "r"(r2), "r"(r3), "r"(smem_u32(bar))
-        : "memory");
-}
 // Same, with an L2 cache policy (e.g. evict-first for data that is streamed once).
 __device__ __forceinline__ void tma_load_4d_hint(void *smem_dst, const CUtensorMap *map, uint64_t *bar,
                                                  int c0, int c1, int c2, int c3, uint64_t policy) {

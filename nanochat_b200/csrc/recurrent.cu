@@ -86,6 +86,42 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float *__restrict
     }
 }
 
+// Groups of up to 512 channels: a warp per group.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) gated_norm_warp_kernel(const float *__restrict__ x, const T *__restrict__ gate,
+                                                              long long gate_stride, const float *__restrict__ w, T *__restrict__ out,
+                                                              long long n, int C, int group, float eps, int gate_silu) {
+    const int lane = threadIdx.x & 31, per_row = C / group;
+    const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (id >= n) return;
+    const long long row = id / per_row;
+    const int c0 = (int)(id - row * per_row) * group;
+    float4 a[NV];
+    Quad<T> g[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (k * 32 + lane) * 4;
+        a[k] = load_quad<true>(x + row * C + c0 + c, c < group, 4).w;
+        g[k] = load_quad<true>(gate + row * gate_stride + c0 + c, c < group, 4);
+        ss = fmaf(a[k].x, a[k].x, fmaf(a[k].y, a[k].y, fmaf(a[k].z, a[k].z, fmaf(a[k].w, a[k].w, ss))));
+    }
+#pragma unroll
+    for (int off = 16; off; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    const float inv = rsqrtf(ss / (float)group + eps);
+    auto gate_of = [&](float z) {
+        return gate_silu ? silu_of<T>(z) : (sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z)));
+    };
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (k * 32 + lane) * 4;
+        if (c >= group) continue;
+        const float4 gf = widen(g[k]), wf = *reinterpret_cast<const float4 *>(w + c0 + c);
+        store_quad<true>(out + row * C + c0 + c, make_float4(a[k].x * inv * wf.x * gate_of(gf.x), a[k].y * inv * wf.y * gate_of(gf.y),
+                                                             a[k].z * inv * wf.z * gate_of(gf.z), a[k].w * inv * wf.w * gate_of(gf.w)), 4);
+    }
+}
+
 template <typename T>
 static cudaError_t gated_norm_launch(const float *x, const T *gate, int64_t gate_stride, const float *w, T *out, int rows, int C,
                                      int group, float eps, int gate_silu, cudaStream_t s) {
@@ -94,6 +130,14 @@ static cudaError_t gated_norm_launch(const float *x, const T *gate, int64_t gate
                      (((uintptr_t)gate | (uintptr_t)out | (uintptr_t)gate_stride * elem) & (4 * elem - 1)) == 0;
     const int per = (group + 1023) / 1024;
     const dim3 grid(rows, C / group);
+    if (vec && group <= 512) {
+        const long long n = (long long)rows * (C / group);
+        const unsigned blocks = (unsigned)((n + 7) / 8);
+        if (group <= 128) gated_norm_warp_kernel<T, 1><<<blocks, 256, 0, s>>>(x, gate, gate_stride, w, out, n, C, group, eps, gate_silu);
+        else if (group <= 256) gated_norm_warp_kernel<T, 2><<<blocks, 256, 0, s>>>(x, gate, gate_stride, w, out, n, C, group, eps, gate_silu);
+        else gated_norm_warp_kernel<T, 4><<<blocks, 256, 0, s>>>(x, gate, gate_stride, w, out, n, C, group, eps, gate_silu);
+        return cudaGetLastError();
+    }
     if (!vec || per > 8) gated_norm_kernel<T, 0><<<grid, 256, 0, s>>>(x, gate, gate_stride, w, out, C, group, eps, gate_silu);
     else if (per <= 1) gated_norm_kernel<T, 1><<<grid, 256, 0, s>>>(x, gate, gate_stride, w, out, C, group, eps, gate_silu);
     else if (per <= 2) gated_norm_kernel<T, 2><<<grid, 256, 0, s>>>(x, gate, gate_stride, w, out, C, group, eps, gate_silu);

@@ -388,10 +388,12 @@ def gated_scan(u, y, gates, gate_bias, y_bias, rate, state, B, T):
     if rows != B * T or y.shape != u.shape or y.dtype != u.dtype or gates.shape != (blocks, rows, 2 * (C // blocks)):
         raise RuntimeError(f"nckv::{name}: shapes do not match ({tuple(u.shape)}, {tuple(y.shape)}, gates {tuple(gates.shape)})")
     out = torch.empty(rows, C, dtype=u.dtype, device=u.device)
+    need = _lib.lib.nckv_gated_scan_workspace_bytes(B, T, C)
+    ws = torch.empty(need, dtype=torch.uint8, device=u.device) if need else None
     idx, stream = _ctx(u)
     with ops._device_guard(idx):
         _lib.call("nckv_gated_scan", _ptr(u), _row_stride(name, u), _ptr(y), _row_stride(name, y), _ptr(gates), _ptr(gate_bias),
-                  _ptr(y_bias), _ptr(rate), _ptr(state), _ptr(out), B, T, C, blocks, int(u.dtype == torch.float32), stream)
+                  _ptr(y_bias), _ptr(rate), _ptr(state), _ptr(out), B, T, C, blocks, int(u.dtype == torch.float32), _ptr(ws), need, stream)
     return out
 
 
@@ -420,10 +422,15 @@ def delta_rule(q, k, v, decay_logits, decay_bias, rate, beta_logits, state, B, T
                       _ptr(state), B, heads, kv_heads, dim, vdim, f32, stream)
         return out
     out = torch.empty(rows, heads * vdim, dtype=torch.float32, device=q.device)
-    need = _lib.lib.nckv_delta_workspace_bytes(B, T, heads, dim)
+    chunks = not f32 and dim <= 128 and T > 4
+    need = (_lib.lib.nckv_delta_chunk_workspace_bytes if chunks else _lib.lib.nckv_delta_workspace_bytes)(B, T, heads, dim)
     ws = torch.empty(need, dtype=torch.uint8, device=q.device)
     with ops._device_guard(idx):
-        _lib.call("nckv_delta_rule", *inputs, _ptr(out), _ptr(state), B, T, heads, kv_heads, dim, vdim, f32, _ptr(ws), need, stream)
+        if chunks:
+            status = ops.workspace(q.device, 1, 1, 1)
+            _lib.call("nckv_delta_chunk", *inputs, _ptr(out), _ptr(state), B, T, heads, kv_heads, dim, vdim, _ptr(ws), need, _ptr(status), stream)
+        else:
+            _lib.call("nckv_delta_rule", *inputs, _ptr(out), _ptr(state), B, T, heads, kv_heads, dim, vdim, f32, _ptr(ws), need, stream)
     return gated_norm(out, gate, norm_weight.repeat(heads), vdim, eps)
 
 
