@@ -192,42 +192,71 @@ struct LeftFrag {  // an accumulator fragment as left operand
     }
 };
 
+// d (16 x 16 tokens) = x times the transpose of a lower triangular 16 x 16 matrix; at: row g, this lane's four places
+__device__ __forceinline__ void small_product(float (&d)[2][4], const LeftFrag &x0, const LeftFrag &x1, const float *at) {
+    const Pair4 b0(*reinterpret_cast<const float4 *>(at)), b1(*reinterpret_cast<const float4 *>(at + 8 * DC_T));
+    float t[9][4];
+#pragma unroll
+    for (int i = 0; i < 9; ++i) t[i][0] = t[i][1] = t[i][2] = t[i][3] = 0.f;
+    mma_tf32(t[0], x0.hi, b0.hi[0], b0.hi[1]);  // tokens 0-7 take nothing from 8-15
+    mma_tf32(t[1], x0.hi, b0.lo[0], b0.lo[1]);
+    mma_tf32(t[2], x0.lo, b0.hi[0], b0.hi[1]);
+    mma_tf32(t[3], x0.hi, b1.hi[0], b1.hi[1]);
+    mma_tf32(t[4], x0.hi, b1.lo[0], b1.lo[1]);
+    mma_tf32(t[5], x0.lo, b1.hi[0], b1.hi[1]);
+    mma_tf32(t[6], x1.hi, b1.hi[2], b1.hi[3]);
+    mma_tf32(t[7], x1.hi, b1.lo[2], b1.lo[3]);
+    mma_tf32(t[8], x1.lo, b1.hi[2], b1.hi[3]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        d[0][e] = t[0][e] + (t[1][e] + t[2][e]);
+        d[1][e] = (t[3][e] + t[6][e]) + ((t[4][e] + t[5][e]) + (t[7][e] + t[8][e]));
+    }
+}
+
 __device__ __forceinline__ void bulk_load(void *smem_dst, const void *src, uint32_t bytes, uint64_t *bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(smem_dst)),
                  "l"(src), "r"(bytes), "r"(smem_u32(bar))
                  : "memory");
 }
 
-// fragment tiles 2 j and 2 j + 1 hold channels 16 j + 4 t + {0, 1} and + {2, 3} in columns 2 t and 2 t + 1
-template <int KP>
+// fragment tiles 2 j and 2 j + 1 hold channels 16 j + 4 t + {0, 1} and + {2, 3} in columns 2 t and 2 t + 1.
+// SPLIT > 1 (few heads): the CTA's SPLIT warps share 16 columns, each holding KP / SPLIT key channels; their
+// partial R and P meet in shared memory, everything else stays apart.
+template <int KP, int SPLIT>
 __global__ void __launch_bounds__(128) delta_chunk_kernel(const DeltaChunkParams p) {
-    constexpr int J = KP / 16, RS = dc_row(KP), REC = dc_record(KP);
+    constexpr int J = KP / 16 / SPLIT, RS = dc_row(KP), REC = dc_record(KP);
+    static_assert(J >= 2 && J % 2 == 0, "the update takes two channel groups at a time");
     extern __shared__ __align__(128) float dc_smem[];
     __shared__ uint64_t bar[DC_RING];
+    __shared__ float4 s_part[SPLIT > 1 ? 2 : 1][SPLIT][4][32];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tg = lane & 3;
+    const int part = SPLIT > 1 ? warp : 0, c0 = part * (KP / SPLIT);  // this warp's first key channel
     const int h = blockIdx.x / p.n_cols, b = blockIdx.y;
-    const int col = ((blockIdx.x % p.n_cols) * (blockDim.x >> 5) + warp) * 16 + g;  // this lane's columns: col, col + 8
+    const int groups = SPLIT > 1 ? 1 : blockDim.x >> 5;
+    const int col = ((blockIdx.x % p.n_cols) * groups + (SPLIT > 1 ? 0 : warp)) * 16 + g;  // this lane's columns: col, col + 8
     const bool on0 = col < p.Dv, on1 = col + 8 < p.Dv;
     const float *src = p.records + ((long long)b * p.H + h) * p.n_chunks * REC;
     auto fetch = [&](int i) {  // by one thread
         mbar_arrive_expect_tx(&bar[i % DC_RING], REC * 4);
         bulk_load(dc_smem + (i % DC_RING) * REC, src + (long long)i * REC, REC * 4, &bar[i % DC_RING]);
     };
+    int fetched = 0;
     if (tid == 0) {
         for (int i = 0; i < DC_RING; ++i) mbar_init(&bar[i], 1);
         fence_mbar_init();
-        for (int i = 0; i < DC_RING && i < p.n_chunks; ++i) fetch(i);
+        for (; fetched < DC_RING && fetched < p.n_chunks; ++fetched) fetch(fetched);
     }
 
     float S[2 * J][4];
-    float *state = p.state + ((long long)b * p.H + h) * p.Dk * p.Dv + col;
+    float *state = p.state + (((long long)b * p.H + h) * p.Dk + c0) * p.Dv + col;
 #pragma unroll
     for (int i = 0; i < 2 * J; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int ch = (i >> 1) * 16 + 4 * tg + (i & 1) * 2 + e;
-            S[i][e] = on0 && ch < p.Dk ? state[(long long)ch * p.Dv] : 0.f;
-            S[i][2 + e] = on1 && ch < p.Dk ? state[(long long)ch * p.Dv + 8] : 0.f;
+            S[i][e] = on0 && c0 + ch < p.Dk ? state[(long long)ch * p.Dv] : 0.f;
+            S[i][2 + e] = on1 && c0 + ch < p.Dk ? state[(long long)ch * p.Dv + 8] : 0.f;
         }
     const __nv_bfloat16 *v = p.v + (long long)b * p.T * p.v_stride + (long long)h * p.Dv + col;
     float *out = p.out + (long long)b * p.T * p.H * p.Dv + (long long)h * p.Dv + col;
@@ -248,108 +277,123 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const DeltaChunkParams
     __syncthreads();
 
     bool failed = false;
-    int i = 0;
-    for (; i < p.n_chunks; ++i) {
+    for (int i = 0; i < p.n_chunks; ++i) {
         int ok = 1;
         if (lane == 0) ok = mbar_wait_bounded(&bar[i % DC_RING], (i / DC_RING) & 1u) ? 1 : 0;
         ok = __shfl_sync(0xffffffffu, ok, 0);
         __syncwarp();
         const float *rec = dc_smem + (i % DC_RING) * REC;
-        if (ok) {
-            // R^T (tokens 0-7, 8-15) and P^T: 16 columns of v by 32 token rows
-            float r[4][4];
+        // A matrix instruction takes longer to finish than to issue: neighbours in the order below add to
+        // different accumulators.
+        // R^T (tokens 0-7, 8-15) and P^T: 16 columns of v by 32 token rows; cross terms summed apart
+        float r[4][4], rc[4][4];
 #pragma unroll
-            for (int m = 0; m < 4; ++m) r[m][0] = r[m][1] = r[m][2] = r[m][3] = 0.f;
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) r[m][e] = rc[m][e] = 0.f;
+        if (ok) {
 #pragma unroll
             for (int j = 0; j < J; ++j) {
                 const LeftFrag a0(S[2 * j]), a1(S[2 * j + 1]);
-                const float *at = rec + g * RS + 16 * j + 4 * tg;
+                const float *at = rec + g * RS + c0 + 16 * j + 4 * tg;
+                const Pair4 bb[4] = {Pair4(*reinterpret_cast<const float4 *>(at)), Pair4(*reinterpret_cast<const float4 *>(at + 8 * RS)),
+                                     Pair4(*reinterpret_cast<const float4 *>(at + 16 * RS)), Pair4(*reinterpret_cast<const float4 *>(at + 24 * RS))};
 #pragma unroll
-                for (int m = 0; m < 4; ++m) {
-                    const Pair4 bb(*reinterpret_cast<const float4 *>(at + m * 8 * RS));
-                    mma_tf32(r[m], a0.hi, bb.hi[0], bb.hi[1]);
-                    mma_tf32(r[m], a1.hi, bb.hi[2], bb.hi[3]);
-                    mma_tf32(r[m], a0.hi, bb.lo[0], bb.lo[1]);
-                    mma_tf32(r[m], a1.hi, bb.lo[2], bb.lo[3]);
-                    mma_tf32(r[m], a0.lo, bb.hi[0], bb.hi[1]);
-                    mma_tf32(r[m], a1.lo, bb.hi[2], bb.hi[3]);
+                for (int m = 0; m < 4; ++m) mma_tf32(r[m], a0.hi, bb[m].hi[0], bb[m].hi[1]);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) mma_tf32(rc[m], a0.hi, bb[m].lo[0], bb[m].lo[1]);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) mma_tf32(r[m], a1.hi, bb[m].hi[2], bb[m].hi[3]);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) mma_tf32(rc[m], a0.lo, bb[m].hi[0], bb[m].hi[1]);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) mma_tf32(rc[m], a1.hi, bb[m].lo[2], bb[m].lo[3]);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) mma_tf32(rc[m], a1.lo, bb[m].hi[2], bb[m].hi[3]);
+            }
+        }
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) r[m][e] += rc[m][e];
+        if (SPLIT > 1) {
+#pragma unroll
+            for (int m = 0; m < 4; ++m) s_part[i & 1][part][m][lane] = make_float4(r[m][0], r[m][1], r[m][2], r[m][3]);
+        }
+        failed = __syncthreads_or(!ok);  // behind it nobody reads the record before this one any more
+        if (failed) break;
+        if (tid == 0 && i > 0 && fetched < p.n_chunks) fetch(fetched++);
+        if (SPLIT > 1) {
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+                if (m >= 2 && part != m - 2) continue;  // warp 0 and 1 answer for the outputs of 8 tokens each
+                r[m][0] = r[m][1] = r[m][2] = r[m][3] = 0.f;
+#pragma unroll
+                for (int w = 0; w < SPLIT; ++w) {  // in the same order in every warp
+                    const float4 f = s_part[i & 1][w][m][lane];
+                    r[m][0] += f.x; r[m][1] += f.y; r[m][2] += f.z; r[m][3] += f.w;
                 }
             }
-            const float *tail = rec + 2 * DC_T * RS + KP * DC_T + KP;
-            float u[2][4];
+        }
+        const float *tail = rec + 2 * DC_T * RS + KP * DC_T + KP;
+        float u[2][4];
 #pragma unroll
-            for (int s = 0; s < 2; ++s)
+        for (int s = 0; s < 2; ++s)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    r[s][e] = to_f(v_raw[s][e]) - r[s][e];
-                    u[s][e] = 0.f;
-                }
-            if (i + 1 < p.n_chunks) load_v(i + 1);
-            // u^T = (v - R)^T T^T and o^T = P^T + u^T Q^T; tokens 0-7 take nothing from 8-15
-            {
-                const LeftFrag d0(r[0]), d1(r[1]);
+            for (int e = 0; e < 4; ++e) r[s][e] = to_f(v_raw[s][e]) - r[s][e];
+        if (i + 1 < p.n_chunks) load_v(i + 1);
+        // u^T = (v - R)^T T^T
+        small_product(u, LeftFrag(r[0]), LeftFrag(r[1]), tail + g * DC_T + 4 * tg);
+        const LeftFrag u0(u[0]), u1(u[1]);
+        // S^T <- S^T diag(c_16) + u^T K, four tiles at a time
+        const float *kt = rec + 2 * DC_T * RS, *cw = kt + KP * DC_T;
 #pragma unroll
-                for (int m = 0; m < 2; ++m) {
-                    const Pair4 bb(*reinterpret_cast<const float4 *>(tail + (8 * m + g) * DC_T + 4 * tg));
-                    mma_tf32(u[m], d0.hi, bb.hi[0], bb.hi[1]);
-                    mma_tf32(u[m], d0.hi, bb.lo[0], bb.lo[1]);
-                    mma_tf32(u[m], d0.lo, bb.hi[0], bb.hi[1]);
-                    if (m == 0) continue;
-                    mma_tf32(u[m], d1.hi, bb.hi[2], bb.hi[3]);
-                    mma_tf32(u[m], d1.hi, bb.lo[2], bb.lo[3]);
-                    mma_tf32(u[m], d1.lo, bb.hi[2], bb.hi[3]);
-                }
-            }
-            const LeftFrag u0(u[0]), u1(u[1]);
+        for (int j = 0; j < J; j += 2) {
+            float (&s0)[4] = S[2 * j], (&s1)[4] = S[2 * j + 1], (&s2)[4] = S[2 * j + 2], (&s3)[4] = S[2 * j + 3];
+            const float4 f = *reinterpret_cast<const float4 *>(cw + c0 + 16 * j + 4 * tg);
+            const float4 f2 = *reinterpret_cast<const float4 *>(cw + c0 + 16 * j + 16 + 4 * tg);
+            s0[0] *= f.x; s0[1] *= f.y; s0[2] *= f.x; s0[3] *= f.y;
+            s1[0] *= f.z; s1[1] *= f.w; s1[2] *= f.z; s1[3] *= f.w;
+            s2[0] *= f2.x; s2[1] *= f2.y; s2[2] *= f2.x; s2[3] *= f2.y;
+            s3[0] *= f2.z; s3[1] *= f2.w; s3[2] *= f2.z; s3[3] *= f2.w;
+            const float *at = kt + (c0 + 16 * j + 4 * (g >> 1) + (g & 1)) * DC_T + 4 * tg;
+            const Pair4 b0(*reinterpret_cast<const float4 *>(at)), b1(*reinterpret_cast<const float4 *>(at + 2 * DC_T)),
+                b2(*reinterpret_cast<const float4 *>(at + 16 * DC_T)), b3(*reinterpret_cast<const float4 *>(at + 18 * DC_T));
+            auto term = [&](const uint32_t (&a)[4], int lo, int at0) {
+                mma_tf32(s0, a, lo ? b0.lo[at0] : b0.hi[at0], lo ? b0.lo[at0 + 1] : b0.hi[at0 + 1]);
+                mma_tf32(s1, a, lo ? b1.lo[at0] : b1.hi[at0], lo ? b1.lo[at0 + 1] : b1.hi[at0 + 1]);
+                mma_tf32(s2, a, lo ? b2.lo[at0] : b2.hi[at0], lo ? b2.lo[at0 + 1] : b2.hi[at0 + 1]);
+                mma_tf32(s3, a, lo ? b3.lo[at0] : b3.hi[at0], lo ? b3.lo[at0 + 1] : b3.hi[at0 + 1]);
+            };
+            term(u0.hi, 0, 0);
+            term(u1.hi, 0, 2);
+            term(u0.hi, 1, 0);
+            term(u1.hi, 1, 2);
+            term(u0.lo, 0, 0);
+            term(u1.lo, 0, 2);
+        }
+        // o^T = P^T + u^T Q^T
+        if (SPLIT == 1 || part < 2) {
+            float o[2][4];
+            small_product(o, u0, u1, tail + DC_T * DC_T + g * DC_T + 4 * tg);
 #pragma unroll
-            for (int m = 0; m < 2; ++m) {
-                const Pair4 bb(*reinterpret_cast<const float4 *>(tail + DC_T * DC_T + (8 * m + g) * DC_T + 4 * tg));
-                mma_tf32(r[2 + m], u0.hi, bb.hi[0], bb.hi[1]);
-                mma_tf32(r[2 + m], u0.hi, bb.lo[0], bb.lo[1]);
-                mma_tf32(r[2 + m], u0.lo, bb.hi[0], bb.hi[1]);
-                if (m == 0) continue;
-                mma_tf32(r[2 + m], u1.hi, bb.hi[2], bb.hi[3]);
-                mma_tf32(r[2 + m], u1.hi, bb.lo[2], bb.lo[3]);
-                mma_tf32(r[2 + m], u1.lo, bb.hi[2], bb.hi[3]);
-            }
-            // S^T <- S^T diag(c_16) + u^T K
-            const float *kt = rec + 2 * DC_T * RS, *cw = kt + KP * DC_T;
-#pragma unroll
-            for (int j = 0; j < J; ++j) {
-                const float4 f = *reinterpret_cast<const float4 *>(cw + 16 * j + 4 * tg);
-                const float d[4] = {f.x, f.y, f.z, f.w};
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    float (&s)[4] = S[2 * j + half];
-                    s[0] *= d[2 * half]; s[1] *= d[2 * half + 1]; s[2] *= d[2 * half]; s[3] *= d[2 * half + 1];
-                    const int ch = 16 * j + 4 * (g >> 1) + 2 * half + (g & 1);
-                    const Pair4 bb(*reinterpret_cast<const float4 *>(kt + ch * DC_T + 4 * tg));
-                    mma_tf32(s, u0.hi, bb.hi[0], bb.hi[1]);
-                    mma_tf32(s, u1.hi, bb.hi[2], bb.hi[3]);
-                    mma_tf32(s, u0.hi, bb.lo[0], bb.lo[1]);
-                    mma_tf32(s, u1.hi, bb.lo[2], bb.lo[3]);
-                    mma_tf32(s, u0.lo, bb.hi[0], bb.hi[1]);
-                    mma_tf32(s, u1.lo, bb.hi[2], bb.hi[3]);
-                }
-            }
-#pragma unroll
-            for (int s = 0; s < 2; ++s)
+            for (int s = 0; s < 2; ++s) {
+                if (SPLIT > 1 && part != s) continue;
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int t = i * DC_T + 8 * s + 2 * tg + e;
-                    if (t < p.T && on0) out[t * out_row] = r[2 + s][e];
-                    if (t < p.T && on1) out[t * out_row + 8] = r[2 + s][2 + e];
+                    if (t < p.T && on0) out[t * out_row] = r[2 + s][e] + o[s][e];
+                    if (t < p.T && on1) out[t * out_row + 8] = r[2 + s][2 + e] + o[s][2 + e];
                 }
+            }
         }
-        failed = __syncthreads_or(!ok);  // also: the record has been read by all warps
-        if (failed) break;
-        if (tid == 0 && i + DC_RING < p.n_chunks) fetch(i + DC_RING);
     }
     if (failed) {
         if (tid == 0) {
             atomicOr(p.status, (int)NCKV_ST_TIMEOUT);
             // copies already issued land before the CTA's memory is released
-            for (int f = i; f < i + DC_RING && f < p.n_chunks; ++f) mbar_wait_bounded(&bar[f % DC_RING], (f / DC_RING) & 1u, 100000000ull);
+            for (int f = fetched > DC_RING ? fetched - DC_RING : 0; f < fetched; ++f)
+                mbar_wait_bounded(&bar[f % DC_RING], (f / DC_RING) & 1u, 100000000ull);
         }
         __syncthreads();
         return;
@@ -359,27 +403,36 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const DeltaChunkParams
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int ch = (j >> 1) * 16 + 4 * tg + (j & 1) * 2 + e;
-            if (on0 && ch < p.Dk) state[(long long)ch * p.Dv] = S[j][e];
-            if (on1 && ch < p.Dk) state[(long long)ch * p.Dv + 8] = S[j][2 + e];
+            if (on0 && c0 + ch < p.Dk) state[(long long)ch * p.Dv] = S[j][e];
+            if (on1 && c0 + ch < p.Dk) state[(long long)ch * p.Dv + 8] = S[j][2 + e];
         }
 }
 
 static int dc_pad(int Dk) { return Dk <= 32 ? 32 : (Dk <= 64 ? 64 : 128); }
 
+template <int KP, int SPLIT> static cudaError_t dc_rule(const DeltaChunkParams &p, int warps, cudaStream_t s) {
+    const int smem = DC_RING * dc_record(KP) * (int)sizeof(float);
+    const cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<KP, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    delta_chunk_kernel<KP, SPLIT><<<dim3(p.H * p.n_cols, p.B), warps * 32, smem, s>>>(p);
+    return cudaGetLastError();
+}
+
 template <int KP> static cudaError_t dc_run(DeltaChunkParams p, cudaStream_t s) {
     delta_chunk_prepare_kernel<KP><<<dim3(p.n_chunks * p.H, p.B), KP, 0, s>>>(p);
-    cudaError_t e = cudaGetLastError();
+    const cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
-    // warps that share a CTA share its records; spread them over the SMs while there are few
+    // few heads: several warps to 16 columns; many: CTAs whose warps share a record between their columns
+    constexpr int MOST = KP / 32;
     const int per_head = (p.Dv + 15) / 16;
+    const long long groups = (long long)p.B * p.H * per_head;
+    p.n_cols = per_head;
+    if (MOST >= 4 && groups * 2 <= 4LL * sm_count()) return dc_rule<KP, MOST >= 4 ? 4 : 1>(p, 4, s);
+    if (MOST >= 2 && groups <= 4LL * sm_count()) return dc_rule<KP, MOST >= 2 ? 2 : 1>(p, 2, s);
     int warps = 1;
     while (warps < 4 && warps < per_head && (long long)p.B * p.H * ((per_head + 2 * warps - 1) / (2 * warps)) >= sm_count()) warps *= 2;
     p.n_cols = (per_head + warps - 1) / warps;
-    const int smem = DC_RING * dc_record(KP) * (int)sizeof(float);
-    e = cudaFuncSetAttribute(delta_chunk_kernel<KP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return e;
-    delta_chunk_kernel<KP><<<dim3(p.H * p.n_cols, p.B), warps * 32, smem, s>>>(p);
-    return cudaGetLastError();
+    return dc_rule<KP, 1>(p, warps, s);
 }
 
 }  // namespace nckv

@@ -11,7 +11,6 @@
 //                         tile is the same for both operands and otherwise free.
 //   expert_plain_kernel   fp32, and sizes without 16-byte rows: 32 x 32 tiles on the fp32 pipe.
 // Many bf16 rows take the tensor-memory form in experts_tc.cu.
-#include <stdlib.h>
 #include "experts.cuh"
 
 namespace nckv {
@@ -307,10 +306,7 @@ static cudaError_t expert_plain(const ExpertParams &p, bool up, cudaStream_t s) 
 }
 
 // pairs above which the tensor-memory form is used
-static int expert_many(int E) {
-    if (const char *v = getenv("NCKV_DEV_MANY")) return atoi(v);
-    return 48 * E > 512 ? 48 * E : 512;
-}
+constexpr int EXPERT_MANY = 32;
 
 }  // namespace nckv
 
@@ -389,7 +385,7 @@ int nckv_experts(const void *a, const void *w, void *out, const int32_t *offsets
         NCKV_CUDA_CHECK(expert_plain<__nv_bfloat16>(p, up, s));
         return NCKV_OK;
     }
-    if (R > expert_many(E)) {
+    if (R > EXPERT_MANY) {
         int rc = NCKV_OK;
         NCKV_CUDA_CHECK(experts_tc(p, up, s, &rc));
         return rc;

@@ -5,9 +5,10 @@
 // factors of an output).  A tile's K runs in steps of 64 through a ring in shared memory (128-byte
 // swizzle).  Roles, connected by mbarriers:
 //   warp 0      moves the weights, and without UP the positions (rows of act), by TMA
-//   warps 6-9   UP: the tokens of a tile lie anywhere in h; these warps fetch them with 16-byte asynchronous copies
+//   warps 6-13  UP: the tokens of a tile lie anywhere in h; these warps fetch them with 16-byte asynchronous copies
 //               into the place the swizzle gives them, so h is never copied into sorted order (a gather by
-//               TMA, four rows per instruction, was three times slower than the products).
+//               TMA, four rows per instruction, was three times slower than the products).  Four of the
+//               warps take the even steps, four the odd ones.
 //   warp 1      one thread issues the products into one of two accumulators
 //   warps 2-5   one thread per position reads the other accumulator, applies the router's weight and the
 //               activation (UP) or finds the pair's place (down), and stores
@@ -20,7 +21,7 @@
 namespace nckv {
 
 constexpr int ET_M = 128, ET_K = 64;
-constexpr int ET_THREADS = 192, ET_GATHER = 128;  // UP has ET_GATHER more
+constexpr int ET_THREADS = 192, ET_GATHER = 256;  // UP has ET_GATHER more, in two halves
 constexpr int ET_MAX_EXPERTS = 1024;
 constexpr int ET_A_BYTES = ET_M * ET_K * 2;
 
@@ -86,7 +87,7 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
         prefetch_tensormap(&map_a);
         prefetch_tensormap(&map_w);
         for (int i = 0; i < STAGES; ++i) {
-            mbar_init(&bar_full[i], UP ? 1 + ET_GATHER / 32 : 1);
+            mbar_init(&bar_full[i], UP ? 1 + ET_GATHER / 64 : 1);
             mbar_init(&bar_free[i], 1);
         }
         for (int i = 0; i < 2; ++i) {
@@ -185,15 +186,16 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
     } else if (UP && warp >= 6) {
         // =============== tokens =====================================================================
         // 8 threads fetch the 128 bytes a token has in a step; a thread serves 8 tokens.  A step is handed over
-        // once the LAG steps behind it have been asked for.
-        constexpr int LAG = STAGES - 1;
-        const int pt = tid - ET_THREADS, chunk = pt & 7, r0 = pt >> 3;
-        uint32_t fill = 0;
+        // once the LAG of its own steps behind it have been asked for.
+        constexpr int LAG = STAGES / 2 - 1;
+        const uint32_t odd = tid >= ET_THREADS + ET_GATHER / 2;
+        const int pt = (tid - ET_THREADS) & (ET_GATHER / 2 - 1), chunk = pt & 7, r0 = pt >> 3;
+        uint32_t fill = 0, mine = 0;  // steps, and those of this half: its step k is number 2 k + odd
         bool ok = true;
-        auto hand_over = [&](uint32_t f) {
+        auto hand_over = [&](uint32_t k) {
             fence_proxy_async_smem();  // this thread's copies, before the products read them
             __syncwarp();
-            if (lane == 0) mbar_arrive(&bar_full[f % STAGES]);
+            if (lane == 0) mbar_arrive(&bar_full[(2 * k + odd) % STAGES]);
         };
         for (int idx = blockIdx.x; idx < total && ok; idx += gridDim.x) {
             if (!cur.seek(s_first, p, n_tiles, idx)) break;
@@ -204,6 +206,7 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
                 src[i] = m < cur.m_hi ? static_cast<const __nv_bfloat16 *>(p.a) + (long long)(p.slot[m] / p.top) * p.K + chunk * 8 : nullptr;
             }
             for (int ks = 0; ks < k_steps; ++ks, ++fill) {
+                if ((fill & 1u) != odd) continue;
                 const uint32_t st = fill % STAGES, round = fill / STAGES;
                 if (round > 0 && !warp_wait(&bar_free[st], (round - 1) & 1u)) {
                     ok = false;
@@ -220,16 +223,17 @@ experts_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_consta
                                      : "memory");
                 }
                 asm volatile("cp.async.commit_group;" ::: "memory");
-                if (fill >= (uint32_t)LAG) {
+                if (mine >= (uint32_t)LAG) {
                     asm volatile("cp.async.wait_group %0;" ::"n"(LAG) : "memory");
-                    hand_over(fill - LAG);
+                    hand_over(mine - LAG);
                 }
+                ++mine;
             }
         }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         if (ok)
-            for (uint32_t f = fill > (uint32_t)LAG ? fill - LAG : 0; f < fill; ++f) hand_over(f);
-        else if (lane == 0 && *abort_flag == 0) timed_out();
+            for (uint32_t k = mine > (uint32_t)LAG ? mine - LAG : 0; k < mine; ++k) hand_over(k);
+        if (!ok && lane == 0 && *abort_flag == 0) timed_out();
         __syncwarp();
     } else {
         // =============== results ====================================================================

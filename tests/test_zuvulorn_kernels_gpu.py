@@ -307,7 +307,7 @@ def test_routing(rows, E, top):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF])
-@pytest.mark.parametrize("rows,E,top,W,ff", [(1, 8, 1, 160, 48), (3, 3, 3, 45, 23), (30, 4, 2, 88, 40), (200, 6, 1, 136, 72), (17, 2, 1, 64, 20),
+@pytest.mark.parametrize("rows,E,top,W,ff", [(1, 8, 1, 160, 48), (3, 3, 3, 45, 23), (30, 4, 2, 88, 40), (200, 6, 1, 136, 72), (17, 2, 1, 64, 24), (32, 1, 1, 72, 40), (17, 2, 1, 64, 20),
                                              (600, 3, 1, 192, 136), (700, 5, 2, 328, 264), (1500, 4, 1, 64, 512)])
 def test_expert_products(dtype, rows, E, top, W, ff):
     h = rand(rows, W, dtype=dtype)
