@@ -60,9 +60,9 @@ template <int BIT, int LEN> __device__ __forceinline__ int scatter_sum(float *o,
 }
 
 template <int KP>
-__global__ void __launch_bounds__(KP) delta_chunk_prepare_kernel(const DeltaChunkParams p) {
+__global__ void __launch_bounds__(KP, 640 / KP) delta_chunk_prepare_kernel(const DeltaChunkParams p) {
     constexpr int NW = KP / 32;
-    __shared__ float s_sum[NW][32], s_pair[2][DC_T][DC_T], s_beta[DC_T], s_scale[2][DC_T];
+    __shared__ float s_sum[DC_T / 2][NW][32], s_pair[DC_T * DC_T], s_beta[DC_T], s_scale[2][DC_T];
     const int c = threadIdx.x, lane = c & 31, warp = c >> 5;
     const int h = blockIdx.x % p.H, chunk = blockIdx.x / p.H, b = blockIdx.y;  // heads fastest: rows are shared in L2
     const int g = h / (p.H / p.G), t0 = chunk * DC_T, n = min(DC_T, p.T - t0);
@@ -91,16 +91,16 @@ __global__ void __launch_bounds__(KP) delta_chunk_prepare_kernel(const DeltaChun
     }
     {
         const int at = scatter_sum<16, 32>(part, lane);
-        s_sum[warp][at] = part[0];
+        s_sum[0][warp][at] = part[0];
     }
     __syncthreads();
     if (c < 32) {
         float s = 0.f;
 #pragma unroll
-        for (int i = 0; i < NW; ++i) s += s_sum[i][c];
+        for (int i = 0; i < NW; ++i) s += s_sum[0][i][c];
         s_scale[c >> 4][c & 15] = (c < DC_T ? rsqrtf((float)p.Dk) : 1.f) / sqrtf(s + 1e-6f);
     }
-    __syncthreads();
+    __syncthreads();  // also: the sums above have been read
 #pragma unroll
     for (int t = 0; t < DC_T; ++t) {
         q[t] *= s_scale[0][t];
@@ -117,26 +117,22 @@ __global__ void __launch_bounds__(KP) delta_chunk_prepare_kernel(const DeltaChun
         }
         rec[2 * DC_T * dc_row(KP) + KP * DC_T + c] = cum;
     }
-    // row t of A and Q: k_i carried to token t, times k_t and q_t, summed over the channels
+    // Row t of A and Q: k_i carried to token t, times k_t and q_t, summed over the channels.  The t + (t + 1) entries
+    // of row t are numbers t^2 .. of 256 (A_ti is t^2 + i, Q_ti is t^2 + t + i); 32 at a time are summed.
     float ki[DC_T];
 #pragma unroll
     for (int t = 0; t < DC_T; ++t) {
 #pragma unroll
-        for (int i = 0; i < DC_T; ++i) {
-            if (i < t) ki[i] *= w[t];
-            else if (i == t) ki[i] = k[i];
-            part[i] = i < t ? k[t] * ki[i] : 0.f;
-            part[DC_T + i] = i <= t ? q[t] * ki[i] : 0.f;
-        }
-        const int at = scatter_sum<16, 32>(part, lane);
-        __syncthreads();  // the sums of the row before have been read
-        s_sum[warp][at] = part[0];
-        __syncthreads();
-        if (c < 32) {
-            float s = 0.f;
+        for (int i = 0; i < t; ++i) ki[i] *= w[t];
+        ki[t] = k[t];
 #pragma unroll
-            for (int i = 0; i < NW; ++i) s += s_sum[i][c];
-            s_pair[c >> 4][t][c & 15] = s;
+        for (int e = 0; e < 2 * t + 1; ++e) {
+            const int at = t * t + e;
+            part[at % 32] = e < t ? k[t] * ki[e] : q[t] * ki[e >= t ? e - t : 0];
+            if (at % 32 == 31) {
+                const int mine = scatter_sum<16, 32>(part, lane);
+                s_sum[at / 32][warp][mine] = part[0];
+            }
         }
     }
     {
@@ -144,6 +140,13 @@ __global__ void __launch_bounds__(KP) delta_chunk_prepare_kernel(const DeltaChun
         float4 *dst = reinterpret_cast<float4 *>(rec + 2 * DC_T * dc_row(KP) + c * DC_T);
 #pragma unroll
         for (int i = 0; i < 4; ++i) dst[i] = make_float4(ki[2 * i], ki[2 * i + 1], ki[8 + 2 * i], ki[9 + 2 * i]);
+    }
+    __syncthreads();
+    for (int i = c; i < DC_T * DC_T; i += KP) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < NW; ++j) s += s_sum[i >> 5][j][i & 31];
+        s_pair[i] = s;
     }
     __syncthreads();
     float *tail = rec + 2 * DC_T * dc_row(KP) + KP * DC_T + KP;
@@ -154,12 +157,15 @@ __global__ void __launch_bounds__(KP) delta_chunk_prepare_kernel(const DeltaChun
             float s = t == c ? 1.f : 0.f;
 #pragma unroll
             for (int i = 0; i < DC_T; ++i)
-                if (i < t) s = fmaf(-s_pair[0][t][i], u[i], s);  // u[i] is zero for i < c
+                if (i < t) s = fmaf(-s_pair[t * t + i], u[i], s);  // u[i] is zero for i < c
             u[t] = s_beta[t] * s;
             tail[t * DC_T + dc_place(c)] = u[t];
         }
     }
-    for (int i = c; i < DC_T * DC_T; i += KP) tail[DC_T * DC_T + (i / DC_T) * DC_T + dc_place(i % DC_T)] = s_pair[1][i / DC_T][i % DC_T];
+    for (int i = c; i < DC_T * DC_T; i += KP) {
+        const int t = i / DC_T, j = i % DC_T;
+        tail[DC_T * DC_T + t * DC_T + dc_place(j)] = j <= t ? s_pair[t * t + t + j] : 0.f;
+    }
 }
 
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {

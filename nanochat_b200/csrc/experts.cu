@@ -1,7 +1,7 @@
 // Mixture of experts: routing, and the experts' products for few rows or any size.
 //
-//   route_kernel          a warp per token picks the `top` largest logits (ties: the lower index) and their
-//                         sigmoids; one CTA counts, sorts by expert and writes the order.
+//   route_kernel          a thread (few experts) or a warp per token picks the `top` largest logits (ties: the lower
+//                         index) and their sigmoids; one CTA counts, sorts by expert and writes the order.
 //   route_pick_kernel,    the same for many tokens: choices and counts first, then positions from a prefix sum
 //   route_place_kernel    and one reservation per CTA and expert.
 //   expert_rows_kernel    bf16, few rows: bound by reading each used expert's weights once.  A CTA takes
@@ -59,6 +59,65 @@ template <int NJ> struct RouteRow {
     }
 };
 
+// The same with a row's logits in one thread, EM at most.
+template <int EM> struct RouteThread {
+    uint32_t key[EM];
+    __device__ __forceinline__ void load(const float *z, int E) {
+#pragma unroll
+        for (int e = 0; e < EM; ++e) {
+            const uint32_t bits = e < E ? __float_as_uint(z[e]) : 0u;
+            key[e] = e < E ? (bits & 0x80000000u ? ~bits : bits | 0x80000000u) : 0u;
+        }
+    }
+    __device__ __forceinline__ int next(float &z) {
+        uint32_t best = key[0];
+        int idx = 0;
+#pragma unroll
+        for (int e = 1; e < EM; ++e)
+            if (key[e] > best) {
+                best = key[e];
+                idx = e;
+            }
+#pragma unroll
+        for (int e = 0; e < EM; ++e)
+            if (e == idx) key[e] = 0u;
+        z = __uint_as_float(best & 0x80000000u ? best & 0x7fffffffu : ~best);
+        return idx;
+    }
+};
+
+// Calls put(pair, expert, logit) for every choice of the rows first, first + step, .. of a CTA or grid: by threads
+// (PER_THREAD experts at most) or by warps (32 NJ at most).
+template <int PER_THREAD, int NJ, typename Put>
+__device__ __forceinline__ void route_rows(const RouteParams &p, int cta, int ctas, Put put) {
+    const int tid = threadIdx.x, lane = tid & 31, NT = blockDim.x;
+    if constexpr (PER_THREAD > 0) {
+        for (int row = cta * NT + tid; row < p.rows; row += ctas * NT) {
+            RouteThread<PER_THREAD> z;
+            z.load(p.logits + (long long)row * p.E, p.E);
+            for (int j = 0; j < p.top; ++j) {
+                float zl;
+                const int el = z.next(zl);
+                put(row * p.top + j, el, zl);
+            }
+        }
+    } else {
+        const int step = ctas * (NT >> 5);
+        RouteRow<NJ> z, ahead;
+        int row = cta * (NT >> 5) + (tid >> 5);
+        if (row < p.rows) z.load(p.logits + (long long)row * p.E, p.E, lane);
+        for (; row < p.rows; row += step) {
+            if (row + step < p.rows) ahead.load(p.logits + (long long)(row + step) * p.E, p.E, lane);
+            for (int j = 0; j < p.top; ++j) {
+                float zl;
+                const int el = z.next(p.E, lane, zl);
+                if (lane == 0) put(row * p.top + j, el, zl);
+            }
+            z = ahead;
+        }
+    }
+}
+
 // exclusive prefix sums of count[0 .. E) by the first warp; the total behind the last
 __device__ __forceinline__ void route_prefix(const int *count, int *first, int E) {
     if (threadIdx.x >= 32) return;
@@ -77,59 +136,54 @@ __device__ __forceinline__ void route_prefix(const int *count, int *first, int E
     if (threadIdx.x == 0) first[E] = carry;
 }
 
-template <int NJ>
+// the next free place of every lane's expert (-1: none wanted), one addition per warp and expert
+__device__ __forceinline__ int route_claim(int *next, int expert, int lane) {
+    const unsigned same = __match_any_sync(0xffffffffu, expert);
+    const int first = __ffs(same) - 1;
+    int at = 0;
+    if (lane == first && expert >= 0) at = atomicAdd(&next[expert], __popc(same));
+    return __shfl_sync(0xffffffffu, at, first) + __popc(same & ((1u << lane) - 1));
+}
+
+template <int PER_THREAD, int NJ>
 __global__ void __launch_bounds__(1024) route_kernel(const RouteParams p) {
     __shared__ int s_count[RT_MAX_EXPERTS], s_first[RT_MAX_EXPERTS + 1];
     __shared__ uint16_t s_choice[RT_ONE_CTA];
-    __shared__ float s_weight[RT_ONE_CTA];
-    const int tid = threadIdx.x, lane = tid & 31, NT = blockDim.x;
+    __shared__ float s_logit[RT_ONE_CTA];
+    const int tid = threadIdx.x, lane = tid & 31, NT = blockDim.x, R = p.rows * p.top;
     for (int e = tid; e < p.E; e += NT) s_count[e] = 0;
+    route_rows<PER_THREAD, NJ>(p, 0, 1, [&](int pair, int expert, float z) {
+        s_choice[pair] = (uint16_t)expert;
+        s_logit[pair] = z;
+    });
     __syncthreads();
-    for (int row = tid >> 5; row < p.rows; row += NT >> 5) {
-        RouteRow<NJ> z;
-        z.load(p.logits + (long long)row * p.E, p.E, lane);
-        for (int j = 0; j < p.top; ++j) {
-            float zl;
-            const int el = z.next(p.E, lane, zl);
-            if (lane == 0) {
-                s_choice[row * p.top + j] = (uint16_t)el;
-                s_weight[row * p.top + j] = 1.f / (1.f + expf(-zl));
-                atomicAdd(&s_count[el], 1);
-            }
-        }
-    }
+    for (int i0 = 0; i0 < R; i0 += NT) route_claim(s_count, i0 + tid < R ? s_choice[i0 + tid] : -1, lane);
     __syncthreads();
     route_prefix(s_count, s_first, p.E);
     __syncthreads();
     for (int e = tid; e <= p.E; e += NT) p.offsets[e] = s_first[e];
     __syncthreads();
-    for (int i = tid; i < p.rows * p.top; i += NT) {
-        const int at = atomicAdd(&s_first[s_choice[i]], 1);
-        p.slot[at] = i;
-        p.scale[at] = s_weight[i];
+    for (int i0 = 0; i0 < R; i0 += NT) {
+        const int i = i0 + tid, at = route_claim(s_first, i < R ? s_choice[i] : -1, lane);
+        if (i < R) {
+            p.slot[at] = i;
+            p.scale[at] = 1.f / (1.f + expf(-s_logit[i]));
+        }
     }
 }
 
-template <int NJ>
+template <int PER_THREAD, int NJ>
 __global__ void __launch_bounds__(256) route_pick_kernel(const RouteParams p) {
     __shared__ int s_count[RT_MAX_EXPERTS];
-    const int tid = threadIdx.x, lane = tid & 31, R = p.rows * p.top;
-    int32_t *counts = p.choice + R;
+    const int tid = threadIdx.x;
+    int32_t *counts = p.choice + p.rows * p.top;
     for (int e = tid; e < p.E; e += 256) s_count[e] = 0;
     __syncthreads();
-    for (int row = blockIdx.x * 8 + (tid >> 5); row < p.rows; row += gridDim.x * 8) {
-        RouteRow<NJ> z;
-        z.load(p.logits + (long long)row * p.E, p.E, lane);
-        for (int j = 0; j < p.top; ++j) {
-            float zl;
-            const int el = z.next(p.E, lane, zl);
-            if (lane == 0) {
-                p.choice[row * p.top + j] = el;
-                p.weight[row * p.top + j] = 1.f / (1.f + expf(-zl));
-                atomicAdd(&s_count[el], 1);
-            }
-        }
-    }
+    route_rows<PER_THREAD, NJ>(p, blockIdx.x, gridDim.x, [&](int pair, int expert, float z) {
+        p.choice[pair] = expert;
+        p.weight[pair] = 1.f / (1.f + expf(-z));
+        atomicAdd(&s_count[expert], 1);
+    });
     __syncthreads();
     for (int e = tid; e < p.E; e += 256)
         if (s_count[e]) atomicAdd(&counts[e], s_count[e]);
@@ -148,15 +202,17 @@ __global__ void __launch_bounds__(256) route_place_kernel(const RouteParams p, i
         for (int e = tid; e <= p.E; e += 256) p.offsets[e] = s_first[e];
     for (int e = tid; e < p.E; e += 256) s_count[e] = 0;
     __syncthreads();
-    for (int i = lo + tid; i < hi; i += 256) atomicAdd(&s_count[p.choice[i]], 1);
+    for (int i0 = lo; i0 < hi; i0 += 256) route_claim(s_count, i0 + tid < hi ? p.choice[i0 + tid] : -1, tid & 31);
     __syncthreads();
     for (int e = tid; e < p.E; e += 256)
         if (s_count[e]) s_first[e] += atomicAdd(&cursors[e], s_count[e]);
     __syncthreads();
-    for (int i = lo + tid; i < hi; i += 256) {
-        const int at = atomicAdd(&s_first[p.choice[i]], 1);
-        p.slot[at] = i;
-        p.scale[at] = p.weight[i];
+    for (int i0 = lo; i0 < hi; i0 += 256) {
+        const int i = i0 + tid, at = route_claim(s_first, i < hi ? p.choice[i] : -1, tid & 31);
+        if (i < hi) {
+            p.slot[at] = i;
+            p.scale[at] = p.weight[i];
+        }
     }
 }
 
@@ -334,11 +390,13 @@ int nckv_route(const float *logits, int32_t *offsets, int32_t *slot, float *scal
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int R = rows * top;
     if (R <= RT_ONE_CTA) {
-        const int threads = 32 * (rows < 4 ? 4 : (rows < 32 ? rows : 32));
-        if (E <= 32) route_kernel<1><<<1, threads, 0, s>>>(p);
-        else if (E <= 64) route_kernel<2><<<1, threads, 0, s>>>(p);
-        else if (E <= 256) route_kernel<8><<<1, threads, 0, s>>>(p);
-        else route_kernel<32><<<1, threads, 0, s>>>(p);
+        const int warps = R > 992 ? 32 : (R + 31) / 32, row_warps = rows < 32 ? rows : 32;
+        if (E <= 8) route_kernel<8, 0><<<1, warps * 32, 0, s>>>(p);
+        else if (E <= 16) route_kernel<16, 0><<<1, warps * 32, 0, s>>>(p);
+        else if (E <= 32) route_kernel<32, 0><<<1, warps * 32, 0, s>>>(p);
+        else if (E <= 64) route_kernel<0, 2><<<1, row_warps * 32, 0, s>>>(p);
+        else if (E <= 256) route_kernel<0, 8><<<1, row_warps * 32, 0, s>>>(p);
+        else route_kernel<0, 32><<<1, row_warps * 32, 0, s>>>(p);
         NCKV_CUDA_CHECK(cudaGetLastError());
         return NCKV_OK;
     }
@@ -349,12 +407,13 @@ int nckv_route(const float *logits, int32_t *offsets, int32_t *slot, float *scal
     p.choice = static_cast<int32_t *>(workspace);
     p.weight = reinterpret_cast<float *>(p.choice + R + 2 * E);
     NCKV_CUDA_CHECK(cudaMemsetAsync(p.choice + R, 0, sizeof(int32_t) * 2 * E, s));
-    int grid = (rows + 7) / 8;
-    if (grid > 4 * sm_count()) grid = 4 * sm_count();
-    if (E <= 32) route_pick_kernel<1><<<grid, 256, 0, s>>>(p);
-    else if (E <= 64) route_pick_kernel<2><<<grid, 256, 0, s>>>(p);
-    else if (E <= 256) route_pick_kernel<8><<<grid, 256, 0, s>>>(p);
-    else route_pick_kernel<32><<<grid, 256, 0, s>>>(p);
+    const int want = E <= 32 ? (rows + 255) / 256 : (rows + 7) / 8, grid = want < 4 * sm_count() ? want : 4 * sm_count();
+    if (E <= 8) route_pick_kernel<8, 0><<<grid, 256, 0, s>>>(p);
+    else if (E <= 16) route_pick_kernel<16, 0><<<grid, 256, 0, s>>>(p);
+    else if (E <= 32) route_pick_kernel<32, 0><<<grid, 256, 0, s>>>(p);
+    else if (E <= 64) route_pick_kernel<0, 2><<<grid, 256, 0, s>>>(p);
+    else if (E <= 256) route_pick_kernel<0, 8><<<grid, 256, 0, s>>>(p);
+    else route_pick_kernel<0, 32><<<grid, 256, 0, s>>>(p);
     NCKV_CUDA_CHECK(cudaGetLastError());
     const int per = (R + sm_count() - 1) / sm_count() < 1024 ? 1024 : (R + sm_count() - 1) / sm_count();
     route_place_kernel<<<(R + per - 1) / per, 256, 0, s>>>(p, per);

@@ -3,7 +3,6 @@
 //   short_conv_kernel   out_t = act(b + sum_j taps[j] (x_(t - K + 1 + j) + b_in)), per channel, zeros before the
 //                       start of a sequence; the last K - 1 inputs of every row are carried in fp32.  A
 //                       thread takes a run of tokens of 4 (or 1) channels, all inputs loaded together.
-//   conv_carry_kernel   the carried inputs after a call of more than one run
 //   gated_scan_kernel   S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with log a_t = -rate r_t and the gates
 //                       r, i = sigmoid(logits + bias); out_t = S_t * gelu_tanh(y_t + b_y).  A thread per channel
 //                       and segment.  Prompts are cut into segments that run side by side: a first pass
@@ -17,7 +16,6 @@ namespace nckv {
 // ------------------------------------------------------------------------------------------------
 // short causal convolution
 // ------------------------------------------------------------------------------------------------
-constexpr int CONV_RUN = 8;
 constexpr int CONV_MAX_TAPS = 16;
 
 struct ShortConvParams {
@@ -78,7 +76,19 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
         }
         put_v(static_cast<T *>(p.out) + ((long long)b * p.T + t0 + i) * p.C + c, o);
     }
-    if (gridDim.y == 1) {  // the only run of its row: nobody else reads the carried inputs
+    if (blockIdx.y > 0) return;
+    // Only the first run reads carried inputs (RUN >= KK - 1 where there are several), so it may replace them.
+    if (gridDim.y > 1) {
+#pragma unroll
+        for (int j = 0; j < KK - 1; ++j) {
+            if (j >= K - 1) break;
+            float last[V];
+            get_v(x + (p.T - (K - 1) + j) * p.x_stride, last);
+#pragma unroll
+            for (int e = 0; e < V; ++e) last[e] += bi[e];
+            put_v(carry + (long long)j * p.C, last);
+        }
+    } else {
 #pragma unroll
         for (int j = 1; j < RUN + KK - 1; ++j) {
             const int keep = j - lack - p.T;  // token t0 - (KK - 1) + j is number `keep` of the K - 1 to carry
@@ -87,37 +97,19 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
     }
 }
 
-// the carried inputs after a call: the last K - 1 of those carried before and the call's own
-template <typename T>
-__global__ void __launch_bounds__(256) conv_carry_kernel(const ShortConvParams p) {
-    const int c = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y;
-    if (c >= p.C) return;
-    const float bias = p.in_bias ? p.in_bias[c] : 0.f;
-    float *carry = p.carry + (long long)b * (p.K - 1) * p.C + c;
-    for (int j = 0; j < p.K - 1; ++j) {  // reads run ahead of writes
-        const int t = p.T - (p.K - 1) + j;
-        carry[(long long)j * p.C] = t >= 0 ? to_f(static_cast<const T *>(p.x)[((long long)b * p.T + t) * p.x_stride + c]) + bias
-                                           : carry[(long long)(j + p.T) * p.C];
-    }
-}
-
-template <typename T, int V, int RUN>
+template <typename T, int V, int KK, int RUN>
 static cudaError_t conv_run(const ShortConvParams &p, cudaStream_t s) {
-    const dim3 grid((p.C + 128 * V - 1) / (128 * V), (p.T + RUN - 1) / RUN, p.B);
-    if (p.K <= 2) short_conv_kernel<T, V, 2, RUN><<<grid, 128, 0, s>>>(p);
-    else if (p.K <= 4) short_conv_kernel<T, V, 4, RUN><<<grid, 128, 0, s>>>(p);
-    else if (p.K <= 8) short_conv_kernel<T, V, 8, RUN><<<grid, 128, 0, s>>>(p);
-    else short_conv_kernel<T, V, CONV_MAX_TAPS, RUN><<<grid, 128, 0, s>>>(p);
+    static_assert(RUN == 1 || RUN >= KK - 1, "one run reads the carried inputs");
+    short_conv_kernel<T, V, KK, RUN><<<dim3((p.C + 128 * V - 1) / (128 * V), (p.T + RUN - 1) / RUN, p.B), 128, 0, s>>>(p);
     return cudaGetLastError();
 }
 
 template <typename T, int V>
 static cudaError_t conv_launch(const ShortConvParams &p, cudaStream_t s) {
-    if (p.T == 1) return conv_run<T, V, 1>(p, s);
-    const cudaError_t e = conv_run<T, V, CONV_RUN>(p, s);
-    if (e != cudaSuccess || p.T <= CONV_RUN || p.K == 1) return e;
-    conv_carry_kernel<T><<<dim3((p.C + 255) / 256, p.B), 256, 0, s>>>(p);
-    return cudaGetLastError();
+    if (p.K <= 2) return p.T == 1 ? conv_run<T, V, 2, 1>(p, s) : conv_run<T, V, 2, 8>(p, s);
+    if (p.K <= 4) return p.T == 1 ? conv_run<T, V, 4, 1>(p, s) : conv_run<T, V, 4, 8>(p, s);
+    if (p.K <= 8) return p.T == 1 ? conv_run<T, V, 8, 1>(p, s) : conv_run<T, V, 8, 8>(p, s);
+    return p.T == 1 ? conv_run<T, V, CONV_MAX_TAPS, 1>(p, s) : conv_run<T, V, CONV_MAX_TAPS, 16>(p, s);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -144,57 +136,77 @@ template <> __device__ __forceinline__ void gated_terms<float>(float zr, float z
     d = sqrtf(-expm1f(2.f * la)) * Fn<float>::sigmoid(zi) * u;
 }
 template <> __device__ __forceinline__ void gated_terms<__nv_bfloat16>(float zr, float zi, float rate, float u, float &a, float &d) {
-    const float la = -rate * Fn<__nv_bfloat16>::sigmoid(zr), x = -2.f * la;
+    // both sigmoids with one reciprocal; the cut changes them below 1e-17 only
+    const float er = 1.f + __expf(fminf(-zr, 40.f)), ei = 1.f + __expf(fminf(-zi, 40.f)), inv = __fdividef(1.f, er * ei);
+    const float la = -rate * (ei * inv), x = -2.f * la;
     a = __expf(la);
     // 1 - e^-x: its series where the difference would cancel (the first term left out is x^6 / 720)
     const float small = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, -1.f / 24.f), 1.f / 6.f), -0.5f), 1.f);
     const float y = x < 0.125f ? small : fmaf(-a, a, 1.f);
-    d = (y > 0.f ? y * rsqrtf(y) : 0.f) * Fn<__nv_bfloat16>::sigmoid(zi) * u;
+    d = (y > 0.f ? y * rsqrtf(y) : 0.f) * (er * inv) * u;
 }
 
-constexpr int SC_SEG = 32;   // tokens per segment
-constexpr int SC_AHEAD = 8;  // tokens whose operands are loaded together
+constexpr int SC_SEG = 32;  // tokens per segment
 
 // SCAN: 0 all tokens of a row from its state (few tokens), 1 a segment's decay product and own contribution,
-// 2 a segment's outputs from its initial state
-template <typename T, int SCAN>
+// 2 a segment's outputs from its initial state.  V consecutive channels per thread, AHEAD tokens loaded together.
+template <typename T, int SCAN, int V, int AHEAD>
 __global__ void __launch_bounds__(128) gated_scan_kernel(const GatedScanParams p) {
-    const int c = blockIdx.x * 128 + threadIdx.x, b = blockIdx.z, seg = blockIdx.y;
+    const int c = (blockIdx.x * 128 + threadIdx.x) * V, b = blockIdx.z, seg = blockIdx.y;
     if (c >= p.C) return;
     const int blk = c / p.n, j = c - blk * p.n;
-    const float br = p.gate_bias[c], bi = p.gate_bias[p.C + c], by = p.y_bias[c], rate = p.rate[c];
-    const long long row0 = (long long)b * p.T;
-    const T *u = static_cast<const T *>(p.u) + row0 * p.u_stride + c, *y = static_cast<const T *>(p.y) + row0 * p.y_stride + c;
-    const float *g = p.gates + ((long long)blk * p.B * p.T + row0) * 2 * p.n + j;
-    T *out = static_cast<T *>(p.out) + row0 * p.C + c;
-    float *part = p.parts + ((long long)b * p.n_seg + seg) * 2 * p.C + c;
+    float br[V], bi[V], by[V], rate[V];
+    get_v(p.gate_bias + c, br);
+    get_v(p.gate_bias + p.C + c, bi);
+    get_v(p.y_bias + c, by);
+    get_v(p.rate + c, rate);
     const int t_begin = SCAN ? seg * SC_SEG : 0, t_end = SCAN ? min(p.T, t_begin + SC_SEG) : p.T;
-    float S = SCAN == 0 ? p.state[(long long)b * p.C + c] : (SCAN == 2 ? part[0] : 0.f), prod = 1.f;
-    for (int t0 = t_begin; t0 < t_end; t0 += SC_AHEAD) {
-        float zr[SC_AHEAD], zi[SC_AHEAD];
-        T uu[SC_AHEAD], yy[SC_AHEAD];
+    const long long row = (long long)b * p.T + t_begin;
+    const T *u = static_cast<const T *>(p.u) + row * p.u_stride + c, *y = static_cast<const T *>(p.y) + row * p.y_stride + c;
+    const float *g = p.gates + ((long long)blk * p.B * p.T + row) * 2 * p.n + j;
+    T *out = static_cast<T *>(p.out) + row * p.C + c;
+    float *part = p.parts + ((long long)b * p.n_seg + seg) * 2 * p.C + c;
+    float S[V], prod[V];
 #pragma unroll
-        for (int i = 0; i < SC_AHEAD; ++i) {
-            const long long t = min(t0 + i, t_end - 1);
-            zr[i] = g[t * 2 * p.n];
-            zi[i] = g[t * 2 * p.n + p.n];
-            uu[i] = u[t * p.u_stride];
-            if (SCAN != 1) yy[i] = y[t * p.y_stride];
-        }
-#pragma unroll
-        for (int i = 0; i < SC_AHEAD; ++i) {
-            if (t0 + i >= t_end) break;
-            float a, d;
-            gated_terms<T>(zr[i] + br, zi[i] + bi, rate, to_f(uu[i]), a, d);
-            S = fmaf(a, S, d);
-            if (SCAN == 1) prod *= a;
-            else put(out + (long long)(t0 + i) * p.C, S * gelu_tanh<T>(to_f(yy[i]) + by));
-        }
+    for (int e = 0; e < V; ++e) {
+        S[e] = 0.f;
+        prod[e] = 1.f;
     }
-    if (SCAN == 0) p.state[(long long)b * p.C + c] = S;
+    if (SCAN == 0) get_v(p.state + (long long)b * p.C + c, S);
+    if (SCAN == 2) get_v(part, S);
+    for (int left = t_end - t_begin; left > 0; left -= AHEAD) {
+        float zr[AHEAD][V], zi[AHEAD][V], uu[AHEAD][V], yy[AHEAD][V];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            if (i < left) {
+                get_v(g + (long long)i * 2 * p.n, zr[i]);
+                get_v(g + (long long)i * 2 * p.n + p.n, zi[i]);
+                get_v(u + i * p.u_stride, uu[i]);
+                if (SCAN != 1) get_v(y + i * p.y_stride, yy[i]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            if (i >= left) break;
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                float a, d;
+                gated_terms<T>(zr[i][e] + br[e], zi[i][e] + bi[e], rate[e], uu[i][e], a, d);
+                S[e] = fmaf(a, S[e], d);
+                if (SCAN == 1) prod[e] *= a;
+                else yy[i][e] = S[e] * gelu_tanh<T>(yy[i][e] + by[e]);
+            }
+            if (SCAN != 1) put_v(out + (long long)i * p.C, yy[i]);
+        }
+        g += (long long)AHEAD * 2 * p.n;
+        u += AHEAD * p.u_stride;
+        y += AHEAD * p.y_stride;
+        out += (long long)AHEAD * p.C;
+    }
+    if (SCAN == 0) put_v(p.state + (long long)b * p.C + c, S);
     if (SCAN == 1) {
-        part[0] = S;
-        part[p.C] = prod;
+        put_v(part, S);
+        put_v(part + p.C, prod);
     }
 }
 
@@ -204,16 +216,17 @@ __global__ void __launch_bounds__(64) gated_join_kernel(const GatedScanParams p)
     if (c >= p.C) return;
     float *part = p.parts + (long long)b * p.n_seg * 2 * p.C + c;
     float S = p.state[(long long)b * p.C + c];
-    for (int s0 = 0; s0 < p.n_seg; s0 += 16) {
-        float own[16], prod[16];
+    constexpr int AHEAD = 32;
+    for (int s0 = 0; s0 < p.n_seg; s0 += AHEAD) {
+        float own[AHEAD], prod[AHEAD];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
+        for (int i = 0; i < AHEAD; ++i) {
             const long long at = (long long)min(s0 + i, p.n_seg - 1) * 2 * p.C;
             own[i] = part[at];
             prod[i] = part[at + p.C];
         }
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
+        for (int i = 0; i < AHEAD; ++i) {
             if (s0 + i >= p.n_seg) break;
             part[(long long)(s0 + i) * 2 * p.C] = S;
             S = fmaf(prod[i], S, own[i]);
@@ -224,17 +237,30 @@ __global__ void __launch_bounds__(64) gated_join_kernel(const GatedScanParams p)
 
 static int scan_segments(int T) { return T <= SC_SEG ? 0 : (T + SC_SEG - 1) / SC_SEG; }
 
-template <typename T>
+template <typename T, int V, int AHEAD>
 static cudaError_t scan_launch(const GatedScanParams &p, cudaStream_t s) {
-    const unsigned cols = (p.C + 127) / 128;
+    const unsigned cols = (p.C + 128 * V - 1) / (128 * V);
     if (p.n_seg == 0) {
-        gated_scan_kernel<T, 0><<<dim3(cols, 1, p.B), 128, 0, s>>>(p);
+        gated_scan_kernel<T, 0, V, AHEAD><<<dim3(cols, 1, p.B), 128, 0, s>>>(p);
         return cudaGetLastError();
     }
-    gated_scan_kernel<T, 1><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
+    gated_scan_kernel<T, 1, V, AHEAD><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
     gated_join_kernel<<<dim3((p.C + 63) / 64, p.B), 64, 0, s>>>(p);
-    gated_scan_kernel<T, 2><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
+    gated_scan_kernel<T, 2, V, AHEAD><<<dim3(cols, p.n_seg, p.B), 128, 0, s>>>(p);
     return cudaGetLastError();
+}
+
+template <typename T>
+static cudaError_t scan_any(const GatedScanParams &p, cudaStream_t s) {
+    const uintptr_t elem = sizeof(T);
+    const uintptr_t a32 = (uintptr_t)p.gates | (uintptr_t)p.gate_bias | (uintptr_t)p.y_bias | (uintptr_t)p.rate | (uintptr_t)p.state |
+                          (uintptr_t)p.parts;
+    const uintptr_t at = (uintptr_t)p.u | (uintptr_t)p.y | (uintptr_t)p.out | (uintptr_t)(p.u_stride | p.y_stride) * elem;
+    // wide accesses where enough threads are left
+    const bool vec = p.n % 4 == 0 && (a32 & 15) == 0 && (at & (4 * elem - 1)) == 0;
+    const bool many = p.n_seg == 0 || (long long)p.B * p.C * p.n_seg >= 4096LL * sm_count();
+    if (vec && many) return scan_launch<T, 4, 4>(p, s);
+    return scan_launch<T, 1, 8>(p, s);
 }
 
 }  // namespace nckv
@@ -248,7 +274,7 @@ int nckv_short_conv(const void *x, int64_t x_stride, const float *taps, const fl
         set_error("short_conv: null pointer argument");
         return NCKV_E_ARG;
     }
-    if (B <= 0 || T <= 0 || C <= 0 || K <= 0 || B > 65535 || T > 65535 * CONV_RUN) {
+    if (B <= 0 || T <= 0 || C <= 0 || K <= 0 || B > 65535 || T > 65535 * 8) {
         set_error("short_conv: size out of range (B=%d T=%d C=%d K=%d)", B, T, C, K);
         return NCKV_E_ARG;
     }
@@ -298,7 +324,7 @@ int nckv_gated_scan(const void *u, int64_t u_stride, const void *y, int64_t y_st
     p.parts = static_cast<float *>(workspace);
     p.B = B; p.T = T; p.C = C; p.n = C / blocks; p.n_seg = scan_segments(T);
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    NCKV_CUDA_CHECK(f32 ? scan_launch<float>(p, s) : scan_launch<__nv_bfloat16>(p, s));
+    NCKV_CUDA_CHECK(f32 ? scan_any<float>(p, s) : scan_any<__nv_bfloat16>(p, s));
     return NCKV_OK;
 }
 

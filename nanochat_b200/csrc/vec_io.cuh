@@ -47,8 +47,8 @@ __device__ __forceinline__ void put_v(__nv_bfloat16 *p, const float (&o)[8]) {
     *reinterpret_cast<uint4 *>(p) = make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
 }
 
-// Elementwise functions in fp32: bf16 activations get the fast intrinsics (a few fp32 ulps), fp32 ones the
-// full-precision functions.
+// Elementwise functions in fp32: bf16 activations get the fast intrinsics (a few fp32 ulps, tanh aside), fp32 ones
+// the full-precision functions.
 template <typename T> struct Fn;
 template <> struct Fn<float> {
     static __device__ __forceinline__ float exp(float x) { return expf(x); }
@@ -60,9 +60,10 @@ template <> struct Fn<__nv_bfloat16> {
     static __device__ __forceinline__ float exp(float x) { return __expf(x); }
     static __device__ __forceinline__ float sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
     static __device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
-    // 1 - 2 / (e^(2z) + 1); the argument is cut where the result is +-1 anyway
-    static __device__ __forceinline__ float tanh(float z) {
-        return 1.f - __fdividef(2.f, __expf(2.f * fminf(fmaxf(z, -15.f), 15.f)) + 1.f);
+    static __device__ __forceinline__ float tanh(float z) {  // 11 bits, more than a bf16 activation holds
+        float r;
+        asm("tanh.approx.f32 %0, %1;" : "=f"(r) : "f"(z));
+        return r;
     }
 };
 // log(1 + e^z) without overflow

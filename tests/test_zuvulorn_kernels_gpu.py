@@ -287,7 +287,8 @@ def test_sink_and_head_gate(kind, T):
 # ------------------------------------------------------------------------------------------------
 # experts
 # ------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("rows,E,top", [(1, 8, 1), (3, 5, 5), (64, 64, 6), (700, 7, 2), (4096, 16, 1), (5000, 40, 3)])
+@pytest.mark.parametrize("rows,E,top", [(1, 8, 1), (3, 5, 5), (64, 64, 6), (256, 16, 4), (33, 30, 3), (9, 300, 8), (700, 7, 2), (4096, 16, 1),
+                                        (5000, 40, 3), (3000, 12, 2), (2500, 25, 1), (700, 200, 4), (1200, 1000, 2)])
 def test_routing(rows, E, top):
     z = rand(rows, E)
     z[0] = 1.5  # ties go to the lower index
