@@ -41,21 +41,29 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
     for (int e = 0; e < V; ++e) bi[e] = bo[e] = 0.f;
     if (p.in_bias) get_v(p.in_bias + c, bi);
     if (p.bias) get_v(p.bias + c, bo);
+    if (t0 >= KK - 1 && t0 + RUN <= p.T) {  // inside the call: nothing stands between the loads
 #pragma unroll
-    for (int j = 0; j < RUN + KK - 1; ++j) {
-        const int t = t0 - (KK - 1) + j;
+        for (int j = 0; j < RUN + KK - 1; ++j) get_v(x + (long long)(t0 - (KK - 1) + j) * p.x_stride, in[j]);
 #pragma unroll
-        for (int e = 0; e < V; ++e) in[j][e] = 0.f;
-        if (j < lack || t >= p.T) continue;
-        if (t >= 0) get_v(x + t * p.x_stride, in[j]);
-        else get_v(carry + (long long)(K - 1 + t) * p.C, in[j]);  // what is carried has its bias already
-    }
+        for (int j = 0; j < RUN + KK - 1; ++j)
 #pragma unroll
-    for (int j = 0; j < RUN + KK - 1; ++j)
-        if (t0 - (KK - 1) + j >= 0) {
+            for (int e = 0; e < V; ++e) in[j][e] = j < lack ? 0.f : in[j][e] + bi[e];
+    } else {
 #pragma unroll
-            for (int e = 0; e < V; ++e) in[j][e] += bi[e];
+        for (int j = 0; j < RUN + KK - 1; ++j) {
+            const int t = t0 - (KK - 1) + j;
+#pragma unroll
+            for (int e = 0; e < V; ++e) in[j][e] = 0.f;
+            if (j < lack || t >= p.T) continue;
+            if (t >= 0) {
+                get_v(x + t * p.x_stride, in[j]);
+#pragma unroll
+                for (int e = 0; e < V; ++e) in[j][e] += bi[e];
+            } else {
+                get_v(carry + (long long)(K - 1 + t) * p.C, in[j]);  // what is carried has its bias already
+            }
         }
+    }
     float w[KK][V];
 #pragma unroll
     for (int j = 0; j < KK; ++j) {
@@ -178,12 +186,11 @@ __global__ void __launch_bounds__(128) gated_scan_kernel(const GatedScanParams p
         float zr[AHEAD][V], zi[AHEAD][V], uu[AHEAD][V], yy[AHEAD][V];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-            if (i < left) {
-                get_v(g + (long long)i * 2 * p.n, zr[i]);
-                get_v(g + (long long)i * 2 * p.n + p.n, zi[i]);
-                get_v(u + i * p.u_stride, uu[i]);
-                if (SCAN != 1) get_v(y + i * p.y_stride, yy[i]);
-            }
+            const long long k = min(i, left - 1);  // past the end: the last token again, not used
+            get_v(g + k * 2 * p.n, zr[i]);
+            get_v(g + k * 2 * p.n + p.n, zi[i]);
+            get_v(u + k * p.u_stride, uu[i]);
+            if (SCAN != 1) get_v(y + k * p.y_stride, yy[i]);
         }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
